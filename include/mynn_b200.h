@@ -339,6 +339,12 @@ int mynn_b200_model_step_device(void *state, void *stream, const int64_t *ids_de
  * (crates/llm/src/session.rs:426-480) without its padding rows.  ids_host int64 [batch, T] (host memory); out_host
  * receives what model() would return for the last position.  T <= max_prefill. */
 int mynn_b200_model_prefill(void *state, const int64_t *ids_host, int T, int past_len, void *out_host);
+/* The same chunk with the logits of chosen rows: rows_host lists n_rows indices b * T + t into the chunk (host memory), out_host
+ * receives [n_rows, vocab]; n_rows = 0 only fills the cache.  Needs output_mode 0 and tp_world 1; at most
+ * max(batch, min(64, batch * max_prefill)) rows per call.  No counterpart in the engine, whose prefill graph returns the last
+ * position only. */
+int mynn_b200_model_prefill_rows(void *state, const int64_t *ids_host, int T, int past_len, const int32_t *rows_host, int n_rows,
+                                 void *out_host);
 /* Fused tensor-parallel reduction over NVLink peer memory (tp_world > 1): each rank exports a 64-byte handle of its
  * shared block; the host gathers the handles in rank order (as it distributes the communicator id) and attaches them
  * before the first step.  The per-layer all-reduce of a decode step (at most 32 rows) then runs as the two fused
@@ -386,6 +392,80 @@ int mynn_b200_tp_dequant_matmul_push(void *stream, const mynn_b200_tp_group *gro
 int mynn_b200_tp_reduce_norm(void *stream, const mynn_b200_tp_group *group, int buffer, void *x, const void *weight, float eps,
                              int M, int dtype, void *workspace, size_t workspace_bytes);
 int mynn_b200_tp_check(void *stream, const mynn_b200_tp_group *group);
+
+/* ---------------------------------------------------------------------------------------------
+ * Block decoders: models given as a list of layers, each with its own sizes, over unquantised weights.  No counterpart in the
+ * engine.  A layer is
+ *     x += residual_mult * LN(mixer(LN(x)));   x += residual_mult * LN(ff(LN(x)))      (ff absent when experts == 0)
+ * with x in f32, LN a layer norm with weight and bias, the mixer causal attention (below) and ff a mixture of SiLU-gated
+ * experts.  Layers [loop_start, loop_stop) run loop_times times in a row with the same weights and a state per pass; before
+ * every pass but the first the embedding output is added to x.  Embedding rows are multiplied by embed_scale; the head is
+ * LN, then a product.  Attention: q/k/v projections through a causal convolution over conv_taps tokens per channel, interleaved
+ * rotation of the first rot_dims dimensions of q and k, scores attn_scale * q.k through softcap * tanh(. / softcap), the last
+ * `window` positions visible.  Experts: softmax router over all experts, groups_keep of `groups` groups by best member, `top`
+ * experts, weights not renormalised.
+ *
+ * They are stepped through the entry points above: configure, model_init, model / model_step_device / model_prefill /
+ * model_prefill_rows, model_destroy.  Logits are f32.  dtype is that of weights, activations and caches; norms, scores, router,
+ * convolution sums and the residual stream are f32 in every dtype.
+ *
+ * initializer order: embed [V, H]; per layer norm1 w, b; norm1b w, b; qkv [heads*dim + kv_heads*(dim+vdim), H]; conv f32
+ *   [taps, rows of qkv] (NULL without); o [H, heads*vdim]; cos, sin f32 [max_seq_len, rot_dims/2] (NULL without); norm2 w, b;
+ *   norm2b w, b; router [experts, H]; gate_up [experts, 2*expert_ff, H] (gate rows, then up rows); down [experts, H, expert_ff]
+ *   (these seven NULL without experts); then final norm w, b; head [V, H].  Norm weights f32.
+ * session_state order: per layer RUN (a repeated layer counts per pass) K ring [batch, kv_heads, cache_rows, dim], V ring
+ *   [batch, kv_heads, cache_rows, vdim], convolution ring [batch, history_rows, rows of qkv] (NULL without), zeroed.  Position p of
+ *   a sequence lives in row p % cache_rows resp. p % history_rows.  cache_rows: a multiple of 128, and at least max_seq_len or
+ *   window - 1 + max_prefill + max_rewind; history_rows >= conv_taps + max_rewind.
+ * past_len of a step is 0 (a new sequence), the number of positions stored, or up to max_rewind fewer than were ever stored. */
+typedef struct mynn_b200_block {
+    int32_t heads, kv_heads, dim, vdim;
+    int32_t conv_taps, rot_dims;
+    int32_t window;  /* 0: the whole past */
+    int32_t cache_rows, history_rows;
+    int32_t experts, expert_ff, top, groups, groups_keep;
+    float attn_scale, softcap; /* softcap 0: none */
+} mynn_b200_block;
+typedef struct mynn_b200_block_model_config {
+    int32_t n_layers, hidden, vocab, max_seq_len, batch, dtype, output_mode, use_graph, max_prefill, max_rewind;
+    int32_t loop_start, loop_stop, loop_times; /* loop_times <= 1: no loop */
+    float embed_scale, residual_mult, norm_eps;
+    const mynn_b200_block *layers;
+} mynn_b200_block_model_config;
+int mynn_b200_model_configure_blocks(const mynn_b200_block_model_config *cfg);
+
+/* The block decoder's operators. */
+/* out = (x - mean) / sqrt(var + eps) * weight + bias per row of x f32 [rows, W]; out in out_dtype. */
+int mynn_b200_layer_norm(void *stream, void *out, const float *x, const float *weight, const float *bias, float eps, int rows, int W,
+                         int out_dtype);
+/* x += mult * LN(sub; post_weight, post_bias) (+ extra, may be NULL); out = LN(x; weight, bias) (may be NULL).  x, extra f32; sub, out
+ * in dtype. */
+int mynn_b200_residual_layer_norm(void *stream, float *x, const void *sub, const float *post_weight, const float *post_bias, float mult,
+                                  const float *extra, const float *weight, const float *bias, void *out, float eps, int rows, int W,
+                                  int dtype);
+/* S new positions *past_dev .. of B sequences: proj [B*S, Hq*D + Hkv*(D+E)] -> causal convolution (f32 [taps, columns of proj]) ->
+ * interleaved rotation -> q_out [B, Hq, S, D] and the rings (see above).  S <= cache_rows. */
+int mynn_b200_short_conv_append(void *stream, void *q_out, void *k_cache, void *v_cache, void *history, const void *proj,
+                                const float *conv, const float *cos_table, const float *sin_table, int B, int S, int Hq, int Hkv, int D,
+                                int E, int taps, int rot_dims, int cache_rows, int history_rows, const int32_t *past_dev, int dtype);
+/* q [B, Hq, Sq, D] at positions active - Sq .. active - 1 over ring caches; out [B, Sq, Hq, E].  window <= 0: the whole past;
+ * softcap <= 0: none.  workspace as for mynn_b200_attention (decode kernel; may be NULL).  plain != 0: the kernel for any sizes. */
+int mynn_b200_window_attention(void *stream, void *out, const void *q, const void *k, const void *v, float scale, float softcap,
+                               int window, int B, int Hq, int Hkv, int Sq, int D, int E, int cache_rows, int active,
+                               const int32_t *active_dev, int dtype, void *workspace, size_t workspace_bytes, int plain);
+/* Expert choice from f32 logits [M, experts]; the workspace (zeroed before its first use) then describes the (token, slot) rows in expert order
+ * for mynn_b200_moe_matmul.  weights_out f32 / experts_out int32 [M, top] may be NULL. */
+size_t mynn_b200_moe_workspace_bytes(int M, int experts, int top);
+int mynn_b200_moe_route(void *stream, void *workspace, size_t workspace_bytes, float *weights_out, int32_t *experts_out, const float *logits,
+                        int M, int experts, int top, int groups, int groups_keep);
+/* out[m, n] = sum_k act[m, k] w[n, k] (w [N, K] in dtype; glu: w [2N, K], out = silu(gate) * up); out_dtype = dtype or f32.
+ * status: device word of the bounded waits (NULL keeps the tensor-core kernel off). */
+int mynn_b200_dense_matmul(void *stream, void *out, const void *act, const void *w, int M, int N, int K, int dtype, int out_dtype, int glu,
+                           int32_t *status);
+/* The same per expert over the M * top routed rows: w [experts, N or 2N, K]; gather: act has one row per token, else one per routed
+ * row.  gather_workspace: M * top * K elements (NULL keeps the tensor-core kernel off when gather is set). */
+int mynn_b200_moe_matmul(void *stream, void *out, const void *act, const void *w, void *route_workspace, void *gather_workspace, int M, int N,
+                         int K, int experts, int top, int gather, int glu, int dtype, int out_dtype, int32_t *status);
 
 /* How many CTAs the 16-bit decode attention kernel lets share the kv rows of one (batch, kv head) pair, given an upper bound
  * of the rows and the number of CTAs of that kernel an SM holds (2 for the ring form at head_dim 128, else 4).  Pure host

@@ -17,11 +17,13 @@
 //     CTA to arrive (atomic ticket, no spinning) combines the partial results and writes the output.
 // Everything else (f32 tensors, head dims other than 64/128, groups larger than 8, more than one query row,
 // causal masks) goes to a generic one-warp-per-query-row kernel that follows the CPU recurrence literally.
+#include <algorithm>
 #include <atomic>
 #include <cstring>
 #include <type_traits>
 
 #include "attention_internal.cuh"
+#include "block_ops.cuh"
 #include "common.cuh"
 #include "i8_gemm.cuh"
 #include "ops_internal.cuh"
@@ -44,7 +46,8 @@ constexpr int kRingDepth = 3;
 __device__ int g_ring_status;  // 31: a wait for a tile ran out of time (read and cleared by mynn_b200_attention_check)
 MYNN_DEFINE_WAIT_BUDGET_SETTER(attention_decode)
 
-template <typename T, int D, bool RING>
+// WIN: a sliding window over a ring cache and a score soft cap (DecodeParams::window, ring_cache, softcap).
+template <typename T, int D, bool RING, bool WIN>
 __global__ void __launch_bounds__(kAttnWarps * 32, RING ? 2 : 4)
 attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const DecodeParams p) {
     constexpr int KS = D / 16;   // k16 steps of QK^T
@@ -56,10 +59,12 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int G = p.G;
     int active = p.active_dev ? *p.active_dev : p.active_host;
-    active = max(0, min(active, p.cache_seq));
+    active = max(0, WIN && p.ring_cache ? active : min(active, p.cache_seq));
+    // rows [lo, active) are seen; the walk starts at the 16-row tile that holds lo (0 without a window)
+    const int lo = WIN ? max(p.window > 0 ? max(0, active - p.window) : 0, p.ring_cache ? active - p.cache_seq : 0) : 0, walk0 = lo & ~15;
     // whole rounds of the CTA's four warps (64 rows): a split that ends inside a round leaves some warps a tile short
-    const int rows_per_split = (((active + p.splits - 1) / p.splits) + 16 * kAttnWarps - 1) / (16 * kAttnWarps) * (16 * kAttnWarps);
-    const int row_beg = split * rows_per_split;
+    const int rows_per_split = (((active - walk0 + p.splits - 1) / p.splits) + 16 * kAttnWarps - 1) / (16 * kAttnWarps) * (16 * kAttnWarps);
+    const int row_beg = walk0 + split * rows_per_split;
     const int row_end = min(row_beg + rows_per_split, active);
 
     const T *kbase = reinterpret_cast<const T *>(p.k) + (size_t)(b * p.Hkv + kvh) * p.cache_seq * D;
@@ -82,12 +87,13 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     uint8_t *ring = ring_raw + (size_t)warp * kRingDepth * kTile;
     const int first = row_beg + 16 * warp;
     const int ntile = first < cache_end ? (cache_end - first + 16 * kAttnWarps - 1) / (16 * kAttnWarps) : 0;
-    const int y0 = (b * p.Hkv + kvh) * p.cache_seq + first;  // tensor row of this warp's first tile
+    const int y0 = (b * p.Hkv + kvh) * p.cache_seq;  // first tensor row of this (batch, kv head)
+    auto slot = [&](int row) { return WIN && p.ring_cache ? row % p.cache_seq : row; };  // a 16-row tile never wraps: both are multiples of 16
     auto issue = [&](int j) {  // lane 0: tile j of this warp into stage j % depth
         if constexpr (RING) {
             const int s = j % kRingDepth;
             uint8_t *st = ring + (size_t)s * kTile;
-            const int y = y0 + 16 * kAttnWarps * j;
+            const int y = y0 + slot(first + 16 * kAttnWarps * j);
             mbar_expect_tx(&full[warp][s], kTile);
 #pragma unroll
             for (int hf = 0; hf < NB; hf++) {
@@ -171,7 +177,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
             for (int e = 0; e < 2; e++) {
                 const int row = base + 8 * nt + 2 * t + e;
-                pv[nt][e] = row < end ? s[nt][e] * p.scale : -INFINITY;
+                const float x = s[nt][e] * p.scale;
+                if constexpr (WIN) pv[nt][e] = row < end && row >= lo ? (p.softcap > 0.f ? fast_soft_cap(x, p.softcap) : x) : -INFINITY;
+                else pv[nt][e] = row < end ? x : -INFINITY;
                 tmax = fmaxf(tmax, pv[nt][e]);
             }
         tmax = fmaxf(tmax, __shfl_xor_sync(0xffffffffu, tmax, 1));
@@ -267,14 +275,14 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         uint4 kr[2][KCH], vr[4][VH];
 #pragma unroll
         for (int nt = 0; nt < 2; nt++) {
-            const T *kp = kbase + (size_t)min(base + 8 * nt + g, last) * D + 8 * t;
+            const T *kp = kbase + (size_t)slot(min(base + 8 * nt + g, last)) * D + 8 * t;
 #pragma unroll
             for (int i = 0; i < KCH; i++) kr[nt][i] = ldg_16(kp + 32 * i);
         }
 #pragma unroll
         for (int r = 0; r < 4; r++) {
             const int row = base + 2 * t + (r & 1) + 8 * (r >> 1);
-            const T *vp = vbase + (size_t)min(row, last) * D + 8 * g;
+            const T *vp = vbase + (size_t)slot(min(row, last)) * D + 8 * g;
 #pragma unroll
             for (int h = 0; h < VH; h++) vr[r][h] = ldg_16(vp + 64 * h);
         }
@@ -456,7 +464,7 @@ static bool decode_ring_possible(int B, int Hkv, int cache_seq) {
 // resident CTAs per SM of the decode kernel: the ring form at head_dim 128 holds 96 KB of tiles per CTA
 static int decode_ctas_per_sm(bool ring, int D) { return ring && D == 128 ? 2 : kAttnCtasPerSm; }
 
-template <typename T, int D>
+template <typename T, int D, bool WIN = false>
 static int launch_decode(cudaStream_t st, const DecodeParams &p, int B, bool ring) {
     CUtensorMap mk, mv;
     memset(&mk, 0, sizeof mk);
@@ -467,7 +475,7 @@ static int launch_decode(cudaStream_t st, const DecodeParams &p, int B, bool rin
         if (int rc = make_map(&mk, p.k, rows, row_bytes, row_bytes, 16)) return rc;
         if (int rc = make_map(&mv, p.v, rows, row_bytes, row_bytes, 16)) return rc;
         constexpr size_t smem = (size_t)kAttnWarps * kRingDepth * 2 * (D / 64) * 16 * 128;
-        auto kern = attention_decode_kernel<T, D, true>;
+        auto kern = attention_decode_kernel<T, D, true, WIN>;
         static bool attr_set = false;
         if (!attr_set) {  // with the kernel's static shared memory every head_dim is past the 48 KB that need no opt-in
             MYNN_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -475,7 +483,7 @@ static int launch_decode(cudaStream_t st, const DecodeParams &p, int B, bool rin
         }
         MYNN_CUDA_OK(launch_pdl(kern, dim3(p.splits, p.Hkv, B), dim3(kAttnWarps * 32), smem, st, mk, mv, p));
     } else {
-        MYNN_CUDA_OK(launch_pdl(attention_decode_kernel<T, D, false>, dim3(p.splits, p.Hkv, B), dim3(kAttnWarps * 32), 0, st, mk, mv, p));
+        MYNN_CUDA_OK(launch_pdl(attention_decode_kernel<T, D, false, WIN>, dim3(p.splits, p.Hkv, B), dim3(kAttnWarps * 32), 0, st, mk, mv, p));
     }
     MYNN_LAUNCH_OK("attention_decode_kernel");
     return MYNN_OK;
@@ -623,6 +631,39 @@ int mynn::launch_attention(cudaStream_t st, void *out, const void *q, const void
     if (int rc = decode_bind_workspace(p, B, D, workspace, workspace_bytes)) return rc;
     if (dtype == MYNN_BF16) return D == 64 ? launch_decode<__nv_bfloat16, 64>(st, p, B, ring) : launch_decode<__nv_bfloat16, 128>(st, p, B, ring);
     return D == 64 ? launch_decode<__half, 64>(st, p, B, ring) : launch_decode<__half, 128>(st, p, B, ring);
+}
+
+// One query row per sequence over a ring cache with a sliding window and a score soft cap (attention_window.cu picks the kernel).
+bool mynn::window_attention_decode_supported(int dtype, const WindowAttention &w) {
+    return w.D == w.E && w.cache_rows % 16 == 0 && w.workspace &&
+           w.workspace_bytes >= mynn_b200_attention_workspace_bytes(w.B, w.Hq, w.Hkv, w.D, w.cache_rows) &&
+           attention_decode_fast_path(w.Sq, w.D, w.Hq, w.Hkv, dtype, w.q, w.k, w.v);
+}
+
+int mynn::launch_window_attention_decode(cudaStream_t st, int dtype, const WindowAttention &w) {
+    if (!window_attention_decode_supported(dtype, w)) return fail(MYNN_E_UNSUPPORTED, "window_attention: not a shape of the decode kernel");
+    DecodeParams p;
+    p.out = w.out;
+    p.q = w.q, p.k = w.k, p.v = w.v;
+    p.scale = w.scale;
+    p.Hq = w.Hq, p.Hkv = w.Hkv, p.G = w.Hq / w.Hkv;
+    p.cache_seq = w.cache_rows;
+    p.active_host = w.active_host;
+    p.active_dev = w.active;
+    int rows_bound = w.active ? w.cache_rows : std::min(w.active_host, w.cache_rows);
+    if (w.window > 0) rows_bound = std::min(rows_bound, w.window + 15);
+    const bool ring = decode_ring_possible(w.B, w.Hkv, w.cache_rows);
+    p.splits = decode_splits(w.B, w.Hkv, rows_bound, 16, decode_ctas_per_sm(ring, w.D));
+    p.k_scale = p.v_scale = nullptr;
+    p.limbs = nullptr;
+    p.ascale = nullptr;
+    p.status = w.status_word;
+    p.window = w.window;
+    p.ring_cache = 1;
+    p.softcap = w.softcap;
+    if (int rc = decode_bind_workspace(p, w.B, w.D, w.workspace, w.workspace_bytes)) return rc;
+    if (dtype == MYNN_BF16) return w.D == 64 ? launch_decode<__nv_bfloat16, 64, true>(st, p, w.B, ring) : launch_decode<__nv_bfloat16, 128, true>(st, p, w.B, ring);
+    return w.D == 64 ? launch_decode<__half, 64, true>(st, p, w.B, ring) : launch_decode<__half, 128, true>(st, p, w.B, ring);
 }
 
 // ------------------------------------------------------------------------------------------------------------

@@ -47,6 +47,9 @@ __device__ __forceinline__ void split_pack(float x, float y, uint32_t &hi, uint3
     lo = (uint32_t)reinterpret_cast<const uint16_t &>(xl) | ((uint32_t)reinterpret_cast<const uint16_t &>(yl) << 16);
 }
 
+// cap * tanh(x / cap) = cap - 2 cap / (1 + e^(2 x / cap)); absolute error a few 1e-7 of cap
+__device__ __forceinline__ float fast_soft_cap(float x, float cap) { return cap - __fdividef(2.0f * cap, 1.0f + __expf(__fdividef(2.0f * x, cap))); }
+
 struct DecodeParams {
     void *out;
     const void *q, *k, *v;
@@ -73,6 +76,10 @@ struct DecodeParams {
     const void *cos_t = nullptr, *sin_t = nullptr;
     const int64_t *fused_pos = nullptr;
     const int32_t *fused_row = nullptr;
+    // Optional (16-bit decode kernel): only the last `window` positions are seen; position p lives in cache row p % cache_seq
+    // (ring_cache: `active` may then exceed cache_seq, which is a multiple of 16); scores pass through a soft cap.
+    int window = 0, ring_cache = 0;
+    float softcap = 0.f;
     int *status = nullptr;  // ring kernel: where a timed-out wait is recorded (null: the library's own word, see attention_check)
 };
 

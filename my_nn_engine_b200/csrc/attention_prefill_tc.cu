@@ -37,6 +37,7 @@
 #include <cstdlib>
 #include <type_traits>
 
+#include "block_ops.cuh"
 #include "common.cuh"
 #include "i8_gemm.cuh"
 #include "ops_internal.cuh"
@@ -61,6 +62,8 @@ struct TcAttnParams {
     int is_causal, out_bshd;
     uint32_t v_lbo, v_sbo;  // byte offsets of the MN-major V descriptor
     int n_qt, heads_per_grid, B;  // 1-D grid: query tiles x (heads or head pairs) x batch, query tile slowest
+    int window, ring_cache;  // WIN kernels: see WindowAttention (block_ops.cuh); cache_seq is a multiple of 128 then
+    float cap2, cap_k;       // soft cap in log2 units: score -> cap2 - 2 cap2 / (1 + 2^(cap_k * raw)); cap2 == 0: none
     int p_tmem;  // probabilities handed to the second product through tensor memory (over the S columns) instead of shared memory
 };
 
@@ -81,6 +84,12 @@ __device__ __forceinline__ uint32_t pack_pair<__half>(float x, float y) {
 __device__ __forceinline__ float fast_exp2(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+__device__ __forceinline__ float fast_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
 
@@ -108,7 +117,7 @@ __device__ __forceinline__ void warp_arrive(uint64_t *bar) {
 }
 
 // grid ceil(Sq / 128) x Hq x B (one dimension), block 320
-template <typename T, int D>
+template <typename T, int D, bool WIN>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, const TcAttnParams p) {
@@ -132,14 +141,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int qt = p.n_qt - 1 - (int)blockIdx.x / per_qt, h = ((int)blockIdx.x % per_qt) % p.heads_per_grid, b = ((int)blockIdx.x % per_qt) / p.heads_per_grid;
     const int kvh = h / (p.Hq / p.Hkv);
     int active = p.active_dev ? *p.active_dev : p.active_host;
-    active = max(0, min(active, p.cache_seq));
+    active = max(0, WIN && p.ring_cache ? active : min(active, p.cache_seq));
     const int q0 = qt * kTcRows;
     const int past = active - p.Sq;
     const int last_row = min(q0 + kTcRows, p.Sq) - 1;
     const int kv_end = p.is_causal ? max(0, min(active, past + last_row + 1)) : active;
-    const int n_tiles = (kv_end + kTcCols - 1) / kTcCols;
+    // WIN: the walk starts at the tile of the first position that the CTA's first row sees
+    const int kv_beg = WIN ? max(p.window > 0 ? past + q0 + 1 - p.window : 0, max(0, p.ring_cache ? active - p.cache_seq : 0)) / kTcCols * kTcCols : 0;
+    const int n_tiles = max(0, kv_end - kv_beg + kTcCols - 1) / kTcCols;
     const int q_row0 = (b * p.Hq + h) * p.Sq + q0;      // row of the Q map
     const int kv_row0 = (b * p.Hkv + kvh) * p.cache_seq;  // row of the K and V maps
+
+    auto tile_slot = [&](int j) { return WIN && p.ring_cache ? (kv_beg + j * kTcCols) % p.cache_seq : kv_beg + j * kTcCols; };
 
     if (threadIdx.x == 0) {
         mbar_init(&q_full, 1);
@@ -182,7 +195,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (u >= 1 && !mbar_wait(&k_empty[s], (u - 1) & 1, &abort_flag)) return false;
                 uint8_t *kb = s_kv + s * kStage;
                 mbar_expect_tx(&k_full[s], kTile);
-                for (int sl = 0; sl < SL; sl++) tma_load_2d(kb + sl * kTcSlab, &map_k, sl * 128, kv_row0 + j * kTcCols, &k_full[s]);
+                for (int sl = 0; sl < SL; sl++) tma_load_2d(kb + sl * kTcSlab, &map_k, sl * 128, kv_row0 + tile_slot(j), &k_full[s]);
                 return true;
             };
             auto load_v = [&](int j) {
@@ -190,7 +203,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (u >= 1 && !mbar_wait(&v_empty[s], (u - 1) & 1, &abort_flag)) return false;
                 uint8_t *vb = s_kv + s * kStage + kTile;
                 mbar_expect_tx(&v_full[s], kTile);
-                for (int sl = 0; sl < SL; sl++) tma_load_2d(vb + sl * kTcSlab, &map_v, sl * 128, kv_row0 + j * kTcCols, &v_full[s]);
+                for (int sl = 0; sl < SL; sl++) tma_load_2d(vb + sl * kTcSlab, &map_v, sl * 128, kv_row0 + tile_slot(j), &v_full[s]);
                 return true;
             };
             bool ok = load_k(0);
@@ -259,11 +272,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t t_lane = tmem_base + ((uint32_t)(quad * 32) << 16);
         const int qi = min(q0 + row, p.Sq - 1);  // rows past Sq repeat the last one; they are not stored
         const int bound = p.is_causal ? min(active, past + qi + 1) : active;
-        const float sl2 = p.scale * 1.4426950408889634f;
+        const int first = WIN && p.window > 0 ? max(0, bound - p.window) : 0;  // this row sees [first, bound)
+        const bool capped = WIN && p.cap2 > 0.f;
+        const float sl2 = capped ? 1.f : p.scale * 1.4426950408889634f;  // capped scores are already in log2 units
         float m_used = -INFINITY, l = 0.f;
         bool ok = true;
         for (int j = 0; j < n_tiles && ok; j++) {
-            const int sb = j & 1, u = j >> 1, kv0 = j * kTcCols, col0 = kv0 + half * HC;
+            const int sb = j & 1, u = j >> 1, kv0 = kv_beg + j * kTcCols, col0 = kv0 + half * HC;
             if (!warp_wait(&s_full[sb], u & 1, &abort_flag)) {
                 if (lane == 0) give_up(5);
                 ok = false;
@@ -277,10 +292,19 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tc_fence_before();
             if (!p.p_tmem) warp_arrive(&s_empty[sb]);  // the rows are in registers: the S buffer may take tile j + 2
 
+            if (capped) {
+#pragma unroll
+                for (int i = 0; i < HC; i++) s[i] = fmaf(-2.f * p.cap2, fast_rcp(1.f + fast_exp2(s[i] * p.cap_k)), p.cap2);
+            }
             if (col0 + HC > bound) {  // only the diagonal and the last tile carry masked columns
 #pragma unroll
                 for (int i = 0; i < HC; i++)
                     if (col0 + i >= bound) s[i] = -INFINITY;
+            }
+            if (WIN && col0 < first) {  // and the tiles at the window's far edge
+#pragma unroll
+                for (int i = 0; i < HC; i++)
+                    if (col0 + i < first) s[i] = -INFINITY;
             }
             float t0 = -INFINITY, t1 = -INFINITY;
 #pragma unroll
@@ -440,7 +464,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 // and the completion of S_t(j+1) tells the softmax warps that O_t(j) is complete as well (they may rescale O_t).
 //
 // grid ceil(Sq / 128) x Hq / 2 x B (one dimension), block 320: warp 0 TMA, warp 1 MMA, warps 2-5 softmax of head 0, warps 6-9 of head 1.
-template <typename T, int D>
+template <typename T, int D, bool WIN>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, const TcAttnParams p) {
@@ -458,13 +482,17 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
     const int qt = p.n_qt - 1 - (int)blockIdx.x / per_qt, h0 = 2 * (((int)blockIdx.x % per_qt) % p.heads_per_grid), b = ((int)blockIdx.x % per_qt) / p.heads_per_grid;
     const int kvh = h0 / (p.Hq / p.Hkv);  // the group size is even: both heads read the same kv head
     int active = p.active_dev ? *p.active_dev : p.active_host;
-    active = max(0, min(active, p.cache_seq));
+    active = max(0, WIN && p.ring_cache ? active : min(active, p.cache_seq));
     const int q0 = qt * kTcRows;
     const int past = active - p.Sq;
     const int last_row = min(q0 + kTcRows, p.Sq) - 1;
     const int kv_end = p.is_causal ? max(0, min(active, past + last_row + 1)) : active;
-    const int n_tiles = (kv_end + kTcCols - 1) / kTcCols;
+    // WIN: the walk starts at the tile of the first position that the CTA's first row sees
+    const int kv_beg = WIN ? max(p.window > 0 ? past + q0 + 1 - p.window : 0, max(0, p.ring_cache ? active - p.cache_seq : 0)) / kTcCols * kTcCols : 0;
+    const int n_tiles = max(0, kv_end - kv_beg + kTcCols - 1) / kTcCols;
     const int kv_row0 = (b * p.Hkv + kvh) * p.cache_seq;
+
+    auto tile_slot = [&](int j) { return WIN && p.ring_cache ? (kv_beg + j * kTcCols) % p.cache_seq : kv_beg + j * kTcCols; };
 
     if (threadIdx.x == 0) {
         mbar_init(&q_full, 1);
@@ -508,7 +536,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 const int s = j & 1, u = j >> 1;
                 if (u >= 1 && !mbar_wait(&empty[s], (u - 1) & 1, &abort_flag)) return false;
                 mbar_expect_tx(&full[s], kTile);
-                for (int sl = 0; sl < SL; sl++) tma_load_2d(base + s * kTile + sl * kTcSlab, map, sl * 128, kv_row0 + j * kTcCols, &full[s]);
+                for (int sl = 0; sl < SL; sl++) tma_load_2d(base + s * kTile + sl * kTcSlab, map, sl * 128, kv_row0 + tile_slot(j), &full[s]);
                 return true;
             };
             bool ok = load(0, s_k, &map_k, k_full, k_empty);
@@ -580,11 +608,13 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
         const uint32_t colS = t * 128, colO = 256 + t * 128;
         const int qi = min(q0 + row, p.Sq - 1);  // rows past Sq repeat the last one; they are not stored
         const int bound = p.is_causal ? min(active, past + qi + 1) : active;
-        const float sl2 = p.scale * 1.4426950408889634f;
+        const int first = WIN && p.window > 0 ? max(0, bound - p.window) : 0;  // this row sees [first, bound)
+        const bool capped = WIN && p.cap2 > 0.f;
+        const float sl2 = capped ? 1.f : p.scale * 1.4426950408889634f;  // capped scores are already in log2 units
         float m_used = -INFINITY, l = 0.f;
         bool ok = true;
         for (int j = 0; j < n_tiles && ok; j++) {
-            const int kv0 = j * kTcCols;
+            const int kv0 = kv_beg + j * kTcCols;
             if (!warp_wait_spin(&s_full[t], j & 1, &abort_flag)) {
                 if (lane == 0) give_up(15);
                 ok = false;
@@ -595,10 +625,19 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
 #pragma unroll
             for (int c = 0; c < kTcCols / 32; c++) tmem_ld32(t_lane + colS + c * 32, reinterpret_cast<uint32_t *>(s) + c * 32);
             tmem_ld_wait();
+            if (capped) {
+#pragma unroll
+                for (int i = 0; i < kTcCols; i++) s[i] = fmaf(-2.f * p.cap2, fast_rcp(1.f + fast_exp2(s[i] * p.cap_k)), p.cap2);
+            }
             if (kv0 + kTcCols > bound) {  // only the diagonal and the last tile carry masked columns
 #pragma unroll
                 for (int i = 0; i < kTcCols; i++)
                     if (kv0 + i >= bound) s[i] = -INFINITY;
+            }
+            if (WIN && kv0 < first) {  // and the tiles at the window's far edge
+#pragma unroll
+                for (int i = 0; i < kTcCols; i++)
+                    if (kv0 + i < first) s[i] = -INFINITY;
             }
             float t0 = -INFINITY, t1 = -INFINITY, t2 = -INFINITY, t3 = -INFINITY;
 #pragma unroll
@@ -721,10 +760,10 @@ bool attention_prefill_tc_supported(int B, int Hq, int Hkv, int Sq, int D, int c
            (long long)B * Hq * Sq < (1LL << 31) && (long long)B * Hkv * cache_seq_len < (1LL << 31);
 }
 
-template <typename T, int D>
+template <typename T, int D, bool WIN>
 static int launch_tc(cudaStream_t st, const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const TcAttnParams &p, int B) {
     constexpr size_t smem = (size_t)(D / 64) * kTcSlab * (1 + 4) + 2 * kTcSlab + 1024;  // Q, 2 x (K, V), P, alignment slack
-    auto kern = attention_prefill_tc_kernel<T, D>;
+    auto kern = attention_prefill_tc_kernel<T, D, WIN>;
     static bool attr_set = false;
     if (!attr_set) {
         MYNN_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -739,10 +778,10 @@ static int launch_tc(cudaStream_t st, const CUtensorMap &mq, const CUtensorMap &
     return MYNN_OK;
 }
 
-template <typename T, int D>
+template <typename T, int D, bool WIN>
 static int launch_tc2(cudaStream_t st, const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const TcAttnParams &p, int B) {
     constexpr size_t smem = (size_t)(D / 64) * kTcSlab * 6 + 1024;  // 2 x Q, 2 x K, 2 x V, alignment slack
-    auto kern = attention_prefill_tc2_kernel<T, D>;
+    auto kern = attention_prefill_tc2_kernel<T, D, WIN>;
     static bool attr_set = false;
     if (!attr_set) {
         MYNN_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
@@ -757,10 +796,33 @@ static int launch_tc2(cudaStream_t st, const CUtensorMap &mq, const CUtensorMap 
     return MYNN_OK;
 }
 
+// the maps, and the kernel for the group size
+template <bool WIN>
+static int launch_maps(cudaStream_t st, TcAttnParams p, const void *q, const void *k, const void *v, int B, int D, int dtype) {
+    // V tile in shared memory: D / 64 slabs of [128 kv rows][64 head-dim elements]: the next 64 head-dim elements are one
+    // slab further (leading offset), the next 8 kv rows 8 x 128 bytes further (stride offset)
+    p.v_lbo = kTcSlab;
+    p.v_sbo = 1024;
+    p.p_tmem = g_prefill_attention_mode == 3;
+    // the maps describe the tensors as bytes: rows of D * 2 bytes, boxes of 128 bytes x 128 rows
+    CUtensorMap mq, mk, mv;
+    const uint64_t row_bytes = (uint64_t)D * 2;
+    if (int rc = make_map(&mq, q, (uint64_t)B * p.Hq * p.Sq, row_bytes, row_bytes, kTcRows)) return rc;
+    if (int rc = make_map(&mk, k, (uint64_t)B * p.Hkv * p.cache_seq, row_bytes, row_bytes, kTcCols)) return rc;
+    if (int rc = make_map(&mv, v, (uint64_t)B * p.Hkv * p.cache_seq, row_bytes, row_bytes, kTcCols)) return rc;
+    // an even group size can put two query heads of one kv head into every CTA (mode 4)
+    if ((p.Hq / p.Hkv) % 2 == 0 && g_prefill_attention_mode == 1) {
+        if (dtype == MYNN_BF16) return D == 64 ? launch_tc2<__nv_bfloat16, 64, WIN>(st, mq, mk, mv, p, B) : launch_tc2<__nv_bfloat16, 128, WIN>(st, mq, mk, mv, p, B);
+        return D == 64 ? launch_tc2<__half, 64, WIN>(st, mq, mk, mv, p, B) : launch_tc2<__half, 128, WIN>(st, mq, mk, mv, p, B);
+    }
+    if (dtype == MYNN_BF16) return D == 64 ? launch_tc<__nv_bfloat16, 64, WIN>(st, mq, mk, mv, p, B) : launch_tc<__nv_bfloat16, 128, WIN>(st, mq, mk, mv, p, B);
+    return D == 64 ? launch_tc<__half, 64, WIN>(st, mq, mk, mv, p, B) : launch_tc<__half, 128, WIN>(st, mq, mk, mv, p, B);
+}
+
 int launch_attention_prefill_tc(cudaStream_t st, void *out, const void *q, const void *k, const void *v, float scale, int B, int Hq,
                                 int Hkv, int Sq, int D, int cache_seq_len, int active_seq_kv, const int32_t *active_seq_kv_dev,
                                 int is_causal, int dtype, int out_bshd) {
-    TcAttnParams p;
+    TcAttnParams p = {};
     p.out = out;
     p.scale = scale;
     p.Hq = Hq;
@@ -771,24 +833,40 @@ int launch_attention_prefill_tc(cudaStream_t st, void *out, const void *q, const
     p.active_dev = active_seq_kv_dev;
     p.is_causal = is_causal;
     p.out_bshd = out_bshd;
-    // V tile in shared memory: D / 64 slabs of [128 kv rows][64 head-dim elements]: the next 64 head-dim elements are one
-    // slab further (leading offset), the next 8 kv rows 8 x 128 bytes further (stride offset)
-    p.v_lbo = kTcSlab;
-    p.v_sbo = 1024;
-    p.p_tmem = g_prefill_attention_mode == 3;
-    // the maps describe the tensors as bytes: rows of D * 2 bytes, boxes of 128 bytes x 128 rows
-    CUtensorMap mq, mk, mv;
-    const uint64_t row_bytes = (uint64_t)D * 2;
-    if (int rc = make_map(&mq, q, (uint64_t)B * Hq * Sq, row_bytes, row_bytes, kTcRows)) return rc;
-    if (int rc = make_map(&mk, k, (uint64_t)B * Hkv * cache_seq_len, row_bytes, row_bytes, kTcCols)) return rc;
-    if (int rc = make_map(&mv, v, (uint64_t)B * Hkv * cache_seq_len, row_bytes, row_bytes, kTcCols)) return rc;
-    // an even group size can put two query heads of one kv head into every CTA (mode 4)
-    if ((Hq / Hkv) % 2 == 0 && g_prefill_attention_mode == 1) {
-        if (dtype == MYNN_BF16) return D == 64 ? launch_tc2<__nv_bfloat16, 64>(st, mq, mk, mv, p, B) : launch_tc2<__nv_bfloat16, 128>(st, mq, mk, mv, p, B);
-        return D == 64 ? launch_tc2<__half, 64>(st, mq, mk, mv, p, B) : launch_tc2<__half, 128>(st, mq, mk, mv, p, B);
+    return launch_maps<false>(st, p, q, k, v, B, D, dtype);
+}
+
+// Several query rows over a ring cache with a sliding window and a score soft cap (attention_window.cu picks the kernel).  A ring of
+// whole 128-row tiles never splits a tile; short chunks are taken as well, a window bounds what their mostly empty tile costs.
+bool window_attention_prefill_supported(int dtype, const WindowAttention &w) {
+    if (g_prefill_attention_mode <= 0 || !tensor_map_api_available()) return false;
+    const bool aligned = (((uintptr_t)w.q | (uintptr_t)w.k | (uintptr_t)w.v | (uintptr_t)w.out) % 16) == 0;
+    return w.Sq >= 16 && w.D == w.E && (w.D == 64 || w.D == 128) && (dtype == MYNN_BF16 || dtype == MYNN_F16) && aligned && w.scale > 0.f &&
+           w.cache_rows % kTcCols == 0 && (long long)w.B * w.Hq * w.Sq >= kTcRows && (long long)w.B * w.Hq * w.Sq < (1LL << 31) &&
+           (long long)w.B * w.Hkv * w.cache_rows < (1LL << 31);
+}
+
+int launch_window_attention_prefill(cudaStream_t st, int dtype, const WindowAttention &w) {
+    if (!window_attention_prefill_supported(dtype, w)) return fail(MYNN_E_UNSUPPORTED, "window_attention: not a shape of the tensor-core prefill kernel");
+    TcAttnParams p = {};
+    p.out = w.out;
+    p.scale = w.scale;
+    p.Hq = w.Hq;
+    p.Hkv = w.Hkv;
+    p.Sq = w.Sq;
+    p.cache_seq = w.cache_rows;
+    p.active_host = w.active_host;
+    p.active_dev = w.active;
+    p.is_causal = 1;
+    p.out_bshd = 1;
+    p.window = w.window;
+    p.ring_cache = 1;
+    if (w.softcap > 0.f) {
+        const float log2e = 1.4426950408889634f;
+        p.cap2 = w.softcap * log2e;
+        p.cap_k = 2.f * w.scale * log2e / w.softcap;
     }
-    if (dtype == MYNN_BF16) return D == 64 ? launch_tc<__nv_bfloat16, 64>(st, mq, mk, mv, p, B) : launch_tc<__nv_bfloat16, 128>(st, mq, mk, mv, p, B);
-    return D == 64 ? launch_tc<__half, 64>(st, mq, mk, mv, p, B) : launch_tc<__half, 128>(st, mq, mk, mv, p, B);
+    return launch_maps<true>(st, p, w.q, w.k, w.v, w.B, w.D, dtype);
 }
 
 // Reads and clears the status word of the tensor-core prefill kernels (the stream must be idle).

@@ -1,0 +1,127 @@
+// Operators of the block decoder (block_model.cu): layer norms with their residual step, the short causal convolution with
+// rotation and append, windowed attention, expert routing, and dense / grouped matrix products over unquantised weights.
+// Every size and constant is a parameter; nothing here knows a particular model.
+#pragma once
+#include <cuda_runtime.h>
+#include <stddef.h>
+#include <stdint.h>
+
+namespace mynn {
+
+// ---- layer_norm.cu ---------------------------------------------------------------------------------------------------
+// One step of the residual stream x (f32 [rows, W]), in this order, every part optional:
+//   x  = embed[ids] * embed_scale                         (embed != null; also copied to x0 when that is given)
+//   x += mult * LN(sub; w1, b1)                           (sub != null: one row of dtype per row of x)
+//        with pair_row: sub := sum_s pair_w[row, s] * sub[pair_row[row, s]]   (combination of routed experts)
+//   x += x0                                               (add_x0)
+//   out = LN(x; w2, b2) in dtype                          (out != null)
+// row_map: rows of `out` are taken from rows row_map[i] of x and x is left alone (head of the model).
+// LN(v; w, b) = (v - mean) / sqrt(var + eps) * w + b in f32, var = mean of the squared deviations; w, b f32 [W].
+struct NormStep {
+    const void *embed = nullptr;
+    const int64_t *ids = nullptr;
+    float embed_scale = 1.f;
+    int vocab = 0;
+    float *x = nullptr, *x0 = nullptr;
+    const void *sub = nullptr;
+    const int32_t *pair_row = nullptr;
+    const float *pair_w = nullptr;
+    int top = 0;
+    const float *w1 = nullptr, *b1 = nullptr, *w2 = nullptr, *b2 = nullptr;
+    float mult = 1.f, eps = 0.f;
+    int add_x0 = 0;
+    void *out = nullptr;
+    const int32_t *row_map = nullptr;
+    int W = 0;
+};
+int launch_norm_step(cudaStream_t st, int dtype, const NormStep &p, int rows);
+
+// ---- short_conv.cu ---------------------------------------------------------------------------------------------------
+// The projection rows of S new tokens of B sequences, proj [B * S, C] with C = Hq*D + G*D + G*E (q, k, v), go through the
+// causal convolution y_t[c] = sum_j w[j, c] u_{t-taps+1+j}[c] (f32 [taps, C]; taps == 0: none), q and k through the interleaved
+// rotation of the first rot_dims dimensions of each head (cos / sin f32 [positions, rot_dims / 2]), and on to
+//   q_out [B, Hq, S, D],  k_cache [B, G, cache_rows, D],  v_cache [B, G, cache_rows, E]  (position p in row p % cache_rows).
+// hist [B, hist_rows, C] keeps the unconvolved projection of the last hist_rows positions (position p in row p % hist_rows,
+// hist_rows >= taps).  The new tokens sit at positions *past .. *past + S - 1; positions before 0 count as zero.
+struct ConvStep {
+    const void *proj = nullptr;
+    void *hist = nullptr;
+    int hist_rows = 0;
+    const float *w = nullptr;
+    int taps = 0;
+    const float *cos_t = nullptr, *sin_t = nullptr;
+    int rot_dims = 0;
+    void *q_out = nullptr, *k_cache = nullptr, *v_cache = nullptr;
+    int cache_rows = 0;
+    int B = 0, S = 0, Hq = 0, G = 0, D = 0, E = 0;
+    const int32_t *past = nullptr;
+};
+int launch_conv_step(cudaStream_t st, int dtype, const ConvStep &p);
+
+// ---- attention_window.cu ---------------------------------------------------------------------------------------------
+// Causal attention over ring caches: query row s of a sequence sits at position *active - Sq + s and sees the `window` positions
+// up to and including its own (window <= 0: all of them); position p is read from cache row p % cache_rows.  Scores are
+// scale * q.k, then softcap * tanh(score / softcap) when softcap > 0.  q [B, Hq, Sq, D]; out [B, Sq, Hq, E].
+struct WindowAttention {
+    void *out = nullptr;
+    const void *q = nullptr, *k = nullptr, *v = nullptr;
+    float scale = 1.f, softcap = 0.f;
+    int window = 0;
+    int B = 0, Hq = 0, Hkv = 0, Sq = 0, D = 0, E = 0, cache_rows = 0;
+    int active_host = 0;               // used when active == null
+    const int32_t *active = nullptr;   // device: positions written so far, the new rows included
+    void *workspace = nullptr;
+    size_t workspace_bytes = 0;
+    int *status_word = nullptr;
+};
+int launch_window_attention(cudaStream_t st, int dtype, const WindowAttention &p);
+// The kernel for any sizes and dtypes, whatever the tuned ones would take.
+int launch_window_attention_plain(cudaStream_t st, int dtype, const WindowAttention &p);
+// Tensor-core forms (attention.cu, attention_prefill_tc.cu); they return MYNN_E_UNSUPPORTED for shapes they do not take.
+bool window_attention_decode_supported(int dtype, const WindowAttention &p);
+int launch_window_attention_decode(cudaStream_t st, int dtype, const WindowAttention &p);
+bool window_attention_prefill_supported(int dtype, const WindowAttention &p);
+int launch_window_attention_prefill(cudaStream_t st, int dtype, const WindowAttention &p);
+
+// ---- moe_route.cu ----------------------------------------------------------------------------------------------------
+// Expert choice of M tokens from f32 logits [M, E]: s = softmax(z); of `groups` equal groups of neighbouring experts the `keep`
+// with the largest member stay; the `top` largest s among their experts are chosen, weight s (not renormalised).  The
+// (token, slot) pairs are then ordered by expert.
+struct MoeRoute {
+    float *pair_w;      // [M, top] weights
+    int32_t *pair_row;  // [M, top] place of the pair in the expert order
+    int32_t *pair_e;    // [M, top] chosen expert
+    int32_t *tok_of;    // [M * top] token of the pair at that place
+    int32_t *off;       // [E + 1] first place of every expert
+    int32_t *active;    // [E] experts with at least one pair
+    int32_t *n_active;  // [1]
+    int32_t *count;     // [E] scratch, zero between calls
+    int32_t *tile_e, *tile_row, *n_tiles;  // tiles of kMoeTileRows places that do not cross experts (tensor-core kernel)
+};
+constexpr int kMoeTileRows = 128;
+size_t moe_route_bytes(int M, int experts, int top);
+MoeRoute moe_route_bind(void *base, int M, int experts, int top);
+int launch_moe_route(cudaStream_t st, const MoeRoute &r, const float *logits, int M, int experts, int top, int groups, int keep);
+
+// ---- dense_gemm.cu / dense_gemm_tc.cu --------------------------------------------------------------------------------
+// out[m, n] = sum_k act[m, k] w[n, k], f32 accumulation, weights in `dtype`, out in out_dtype.
+//   glu:      w holds 2 N rows (N gate rows, then N up rows); out[m, n] = silu(gate) * up
+//   experts:  w holds `experts` such blocks; the rows are the (token, slot) places of `route`, place r of expert e is multiplied
+//             with block e; gather: its activation row is tok_of[r], else r.  M is then the number of TOKENS and out has
+//             M * top rows.
+struct DenseGemm {
+    void *out = nullptr;
+    const void *act = nullptr, *w = nullptr;
+    int M = 0, N = 0, K = 0;
+    int out_dtype = 0;
+    int glu = 0;
+    const MoeRoute *route = nullptr;
+    int experts = 1, top = 1, gather = 0;
+    void *gather_ws = nullptr;  // [M * top, K] of dtype: sorted copy of the gathered rows (tensor-core kernel only)
+    int *status = nullptr;      // status word of the bounded waits (tensor-core kernel only)
+};
+int launch_dense_gemm(cudaStream_t st, int dtype, const DenseGemm &g);
+bool dense_gemm_tc_supported(int dtype, const DenseGemm &g);
+int launch_dense_gemm_tc(cudaStream_t st, int dtype, const DenseGemm &g);
+
+}  // namespace mynn

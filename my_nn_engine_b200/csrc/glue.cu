@@ -659,6 +659,21 @@ extern "C" int mynn_b200_embed_gather_dequant(void *stream, void *out, const int
     return MYNN_OK;
 }
 
+namespace mynn {
+// out row i = x row rows[i]; 4-byte words, grid = rows
+__global__ void __launch_bounds__(256) gather_rows_kernel(uint32_t *out, const uint32_t *x, const int32_t *rows, int words) {
+    const uint32_t *src = x + (size_t)rows[blockIdx.x] * words;
+    uint32_t *dst = out + (size_t)blockIdx.x * words;
+    for (int i = threadIdx.x; i < words; i += blockDim.x) dst[i] = src[i];
+}
+int launch_gather_rows(cudaStream_t st, void *out, const void *x, const int32_t *rows_dev, int rows, size_t row_bytes) {
+    if (row_bytes % 4) return fail(MYNN_E_UNSUPPORTED, "gather_rows: rows of %zu bytes", row_bytes);
+    gather_rows_kernel<<<rows, 256, 0, st>>>((uint32_t *)out, (const uint32_t *)x, rows_dev, (int)(row_bytes / 4));
+    MYNN_LAUNCH_OK("gather_rows_kernel");
+    return MYNN_OK;
+}
+}  // namespace mynn
+
 extern "C" int mynn_b200_argmax_last(void *stream, int32_t *out_idx, const void *logits, int rows, int V, int dtype) {
     if (rows < 0 || V <= 0) return fail(MYNN_E_ARG, "argmax_last: bad shape rows=%d V=%d", rows, V);
     if (rows == 0) return MYNN_OK;

@@ -22,6 +22,7 @@
 #include "comm.cuh"
 #include "common.cuh"
 #include "i8_gemm.cuh"
+#include "model_internal.cuh"
 #include "ops_internal.cuh"
 #include "tp_fused.cuh"
 
@@ -29,62 +30,9 @@ extern "C" void model_destroy(void *state);
 
 namespace mynn {
 
-struct LayerW {
-    const void *ln1, *ln2;
-    const int8_t *wq, *wk, *wv, *wo, *wg, *wu, *wd;
-    const void *sq, *sk, *sv, *so, *sg, *su, *sd;
-    void *kc, *vc;
-    void *ksc, *vsc;  // per-token scales of an int8 cache
-    bool qkv_fused, gu_fused;
-};
-
-struct Model {
-    mynn_b200_model_config c;
-    int Hq, Hkv, ffn, vocab_l;  // per-rank sizes
-    int max_rows;               // batch * max(1, max_prefill)
-    std::vector<LayerW> layers;
-    const int8_t *embed;
-    const void *embed_scale, *final_norm, *lm_scale, *cos_t, *sin_t;
-    const int8_t *lm_w;
-    // device buffers
-    char *arena = nullptr;
-    // step inputs, contiguous so that one host-to-device copy delivers them: {past, active, pos0, ids[rows]}
-    int32_t *past_dev, *active_dev;
-    int64_t *pos0_dev, *ids_dev;
-    int64_t *pos_dev;  // positions of a prefill chunk
-    int32_t *tok_dev;
-    char *h_in = nullptr;  // pinned mirror of the input block
-    int *h_status = nullptr;  // pinned: status words of the GEMM workspace and of the tensor-parallel block, fetched with the result
-    void *x, *n, *qkv, *q_rot, *attn, *gu, *h, *last_x, *logits, *logits_full;
-    float *part, *pairs, *pairs_all;  // part = f32 partial sums of a row-parallel product (tp_world > 1, ncclAllReduce path)
-    char *tp_block = nullptr;         // cudaMalloc'd block shared with the peers (fused reduction of decode steps, tp_fused.cuh)
-    size_t tp_block_bytes = 0;
-    TpPeers tp = {};
-    bool tp_attached = false;
-    bool weights_aligned = false;  // every projection weight is 16-byte aligned (the TMA-fed kernels can take all of them)
-    void *attn_ws, *gemm_ws;
-    size_t attn_ws_bytes, gemm_ws_bytes;
-    // streaming (sink + ring) cache: per-slot key positions and the scratch that holds one layer's rotated keys
-    int64_t *kvpos_dev = nullptr;
-    void *k_rot = nullptr;
-    void *k_deq = nullptr, *v_deq = nullptr;  // int8 cache: 16-bit copy of one layer's live rows for the tensor-core prefill attention
-    cudaGraphExec_t stream_graph_exec = nullptr;
-    bool tc_attention_ran = false;  // the step just enqueued went through the tcgen05 prefill attention (its status word is checked)
-    cudaStream_t stream = nullptr;
-    cudaGraphExec_t graph_exec = nullptr;
-};
-
 static mynn_b200_model_config g_cfg;
-static bool g_cfg_set = false;
+static bool g_cfg_set = false, g_cfg_blocks = false;
 static int g_status = MYNN_OK;
-
-static size_t up256(size_t x) { return (x + 255) / 256 * 256; }
-
-#define RC(expr)            \
-    do {                    \
-        int rc__ = (expr);  \
-        if (rc__) return rc__; \
-    } while (0)
 
 // DequantMatMul over any number of rows: the streaming kernel takes up to 32 rows per pass.
 static int gemm(cudaStream_t st, const Model &m, void *out, const void *act, const int8_t *w, const void *scale,
@@ -127,7 +75,9 @@ static int gemm_prequant2(cudaStream_t st, const Model &m, void *out, const int8
 // When the step has at most 32 rows and the int8 tensor-core GEMM is enabled, RMSNorm and Swish*Mul write their
 // (rounded) outputs directly as activation limbs into the GEMM workspace, so no separate pre-pass runs for the
 // q/k/v, gate/up, down and lm_head products.
-static int enqueue_forward(Model &m, cudaStream_t st, int S) {
+// head_rows > 0: logits of the rows listed in rows_dev instead of every sequence's last one; < 0: no logits.
+static int enqueue_forward(Model &m, cudaStream_t st, int S, int head_rows = 0) {
+    if (m.blocks) return block_forward(m, st, S, head_rows);
     const mynn_b200_model_config &c = m.c;
     const int B = c.batch, H = c.hidden, D = c.head_dim, dt = c.dtype;
     const int M = B * S;
@@ -327,22 +277,27 @@ static int enqueue_forward(Model &m, cudaStream_t st, int S) {
             else RC(norm(next_norm, m.part, M, m.x));
         }
     }
-    // --- head: only the last token of each sequence is needed ---
+    if (head_rows < 0) return MYNN_OK;
+    // --- head: only the last token of each sequence is needed, or the rows asked for ---
+    const int R = head_rows > 0 ? head_rows : B;
     const void *xl = m.x;
-    if (S > 1) {
+    if (head_rows > 0) {
+        RC(launch_gather_rows(st, m.last_x, m.x, m.rows_dev, R, (size_t)H * esz));
+        xl = m.last_x;
+    } else if (S > 1) {
         MYNN_CUDA_OK(cudaMemcpy2DAsync(m.last_x, (size_t)H * esz, (const char *)m.x + (size_t)(S - 1) * H * esz,
                                        (size_t)S * H * esz, (size_t)H * esz, B, cudaMemcpyDeviceToDevice, st));
         xl = m.last_x;
     }
-    const bool fused_head = m.gemm_ws != nullptr && B <= kI8MaxRows && H % 16 == 0 && (size_t)H * 4 <= 200 * 1024;
-    if (reduced_limbs) {  // the last fused reduction applied the final norm and left its limbs
-        RC(gemm_prequant(st, m, m.logits, m.lm_w, m.lm_scale, nullptr, B, m.vocab_l, H, dt));
+    const bool fused_head = m.gemm_ws != nullptr && R <= kI8MaxRows && H % 16 == 0 && (size_t)H * 4 <= 200 * 1024;
+    if (reduced_limbs && head_rows == 0) {  // the last fused reduction applied the final norm and left its limbs
+        RC(gemm_prequant(st, m, m.logits, m.lm_w, m.lm_scale, nullptr, R, m.vocab_l, H, dt));
     } else if (fused_head) {
-        RC(launch_rms_norm_limbs(st, dt, m.gemm_ws, m.gemm_ws_bytes, nullptr, nullptr, xl, nullptr, m.final_norm, c.rms_eps, B, H));
-        RC(gemm_prequant(st, m, m.logits, m.lm_w, m.lm_scale, nullptr, B, m.vocab_l, H, dt));
+        RC(launch_rms_norm_limbs(st, dt, m.gemm_ws, m.gemm_ws_bytes, nullptr, nullptr, xl, nullptr, m.final_norm, c.rms_eps, R, H));
+        RC(gemm_prequant(st, m, m.logits, m.lm_w, m.lm_scale, nullptr, R, m.vocab_l, H, dt));
     } else {
-        RC(mynn_b200_rms_norm(st, m.n, xl, m.final_norm, c.rms_eps, B, H, dt));
-        RC(gemm(st, m, m.logits, m.n, m.lm_w, m.lm_scale, nullptr, B, m.vocab_l, H, dt));
+        RC(mynn_b200_rms_norm(st, m.n, xl, m.final_norm, c.rms_eps, R, H, dt));
+        RC(gemm(st, m, m.logits, m.n, m.lm_w, m.lm_scale, nullptr, R, m.vocab_l, H, dt));
     }
     if (c.output_mode == 1) {
         if (tp == 1) {
@@ -360,11 +315,35 @@ static int enqueue_forward(Model &m, cudaStream_t st, int S) {
     return MYNN_OK;
 }
 
+// Stream, pinned blocks and the end of initialisation, common to every graph (the arena and its zero fill are enqueued already).
+static int finish_create(Model *m) {
+    cudaError_t e = cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking);
+    if (e == cudaSuccess) e = cudaMallocHost((void **)&m->h_in, 16 + (size_t)m->max_rows * 8);
+    if (e == cudaSuccess) e = cudaMallocHost((void **)&m->h_status, 2 * sizeof(int));
+    // the zero fills ran on the legacy stream, the model's stream does not wait for it implicitly: finish them before the
+    // first step and before a peer can map a shared block
+    if (e == cudaSuccess) e = cudaDeviceSynchronize();
+    if (e != cudaSuccess) return fail(MYNN_E_CUDA, "model_init: stream / pinned buffer creation failed: %s", cudaGetErrorString(e));
+    return MYNN_OK;
+}
+
 static int model_create(Model **out, void **initializer, void **session_state) {
     if (!g_cfg_set) return fail(MYNN_E_STATE, "model_init: call mynn_b200_model_configure first");
     if (!initializer || !session_state) return fail(MYNN_E_ARG, "model_init: null pointer table");
     Model *m = new Model();
     m->c = g_cfg;
+    m->logits_dtype = g_cfg.dtype;
+    if (g_cfg_blocks) {
+        m->max_rows = m->c.batch * std::max(m->c.max_prefill, 1);
+        int rc = block_create(*m, initializer, session_state);
+        if (!rc) rc = finish_create(m);
+        if (rc) {
+            model_destroy(m);
+            return rc;
+        }
+        *out = m;
+        return MYNN_OK;
+    }
     const mynn_b200_model_config &c = m->c;
     const int tp = c.tp_world;
     m->Hq = c.n_heads / tp;
@@ -423,6 +402,8 @@ static int model_create(Model **out, void **initializer, void **session_state) {
 
     // ---- activation arena ----
     const size_t R = m->max_rows;
+    m->head_capacity = prefill > 1 && tp == 1 ? std::max(c.batch, std::min(64, m->max_rows)) : c.batch;
+    const size_t HR = m->head_capacity;
     const size_t nqkv = (size_t)(m->Hq + 2 * m->Hkv) * D;
     m->attn_ws_bytes = mynn_b200_attention_workspace_bytes(c.batch, m->Hq, m->Hkv, D, c.max_seq_len);
     {
@@ -435,8 +416,8 @@ static int model_create(Model **out, void **initializer, void **session_state) {
     auto take = [&](size_t bytes) { size_t o = off; off += up256(bytes); return o; };
     const size_t o_in = take(16 + R * 8), o_pos = take((size_t)prefill * 8), o_tok = take((size_t)c.batch * 4), o_x = take(R * H * esz), o_n = take(R * H * esz),
                  o_qkv = take(R * nqkv * esz), o_qrot = take(R * m->Hq * D * esz), o_attn = take(R * m->Hq * D * esz),
-                 o_gu = take(R * 2 * m->ffn * esz), o_h = take(R * m->ffn * esz), o_last = take((size_t)c.batch * H * esz),
-                 o_logits = take((size_t)c.batch * m->vocab_l * esz),
+                 o_gu = take(R * 2 * m->ffn * esz), o_h = take(R * m->ffn * esz), o_last = take(HR * H * esz), o_rows = take(HR * 4),
+                 o_logits = take(HR * m->vocab_l * esz),
                  o_full = take(tp > 1 ? (size_t)c.batch * c.vocab * esz : 0), 
                  o_pairs = take((size_t)c.batch * 8), o_pairs_all = take((size_t)c.batch * 8 * std::max(tp, 16)),
                  o_ws = take(m->attn_ws_bytes), o_gws = take(m->gemm_ws_bytes), o_part = take(tp > 1 ? R * H * 4 : 0),
@@ -460,6 +441,7 @@ static int model_create(Model **out, void **initializer, void **session_state) {
     m->tok_dev = (int32_t *)(a + o_tok);
     m->x = a + o_x; m->n = a + o_n; m->qkv = a + o_qkv; m->q_rot = a + o_qrot; m->attn = a + o_attn;
     m->gu = a + o_gu; m->h = a + o_h; m->last_x = a + o_last; m->logits = a + o_logits;
+    m->rows_dev = (int32_t *)(a + o_rows);
     m->logits_full = a + o_full; m->pairs = (float *)(a + o_pairs);
     m->pairs_all = (float *)(a + o_pairs_all); m->attn_ws = a + o_ws;
     m->gemm_ws = m->gemm_ws_bytes ? a + o_gws : nullptr;
@@ -483,20 +465,9 @@ static int model_create(Model **out, void **initializer, void **session_state) {
         m->tp.world = tp;
         m->tp.blocks[c.tp_rank] = m->tp_block;
     }
-    e = cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking);
-    if (e == cudaSuccess) e = cudaMallocHost((void **)&m->h_in, 16 + R * 8);
-    if (e == cudaSuccess) e = cudaMallocHost((void **)&m->h_status, 2 * sizeof(int));
-    if (e != cudaSuccess) {
-        cudaFree(m->arena);
-        delete m;
-        return fail(MYNN_E_CUDA, "model_init: stream / pinned buffer creation failed: %s", cudaGetErrorString(e));
-    }
-    // the zero fills above ran on the legacy stream, the model's stream does not wait for it implicitly: finish them before the
-    // first step and before a peer can map the shared block
-    e = cudaDeviceSynchronize();
-    if (e != cudaSuccess) {
+    if (int rc = finish_create(m)) {
         model_destroy(m);
-        return fail(MYNN_E_CUDA, "model_init: %s", cudaGetErrorString(e));
+        return rc;
     }
     *out = m;
     return MYNN_OK;
@@ -528,23 +499,13 @@ static const void *result_ptr(const Model &m, size_t *bytes) {
         *bytes = (size_t)m.c.batch * 4;
         return m.tok_dev;
     }
-    *bytes = (size_t)m.c.batch * m.c.vocab * dtype_size(m.c.dtype);
+    *bytes = (size_t)m.c.batch * m.c.vocab * dtype_size(m.logits_dtype);
     return m.c.tp_world > 1 ? m.logits_full : m.logits;
 }
 
-// tp > 1 logits arrive as [rank][batch][vocab/tp]; reorder on the host side of the copy.
-static int copy_result_to_host(Model &m, void *dst) {
-    size_t bytes;
-    const void *src = result_ptr(m, &bytes);
-    if (m.c.output_mode == 0 && m.c.tp_world > 1) {
-        const size_t row = (size_t)m.vocab_l * dtype_size(m.c.dtype);
-        for (int r = 0; r < m.c.tp_world; r++)
-            MYNN_CUDA_OK(cudaMemcpy2DAsync((char *)dst + r * row, row * m.c.tp_world, (const char *)src + (size_t)r * m.c.batch * row,
-                                           row, row, m.c.batch, cudaMemcpyDeviceToHost, m.stream));
-    } else {
-        MYNN_CUDA_OK(cudaMemcpyAsync(dst, src, bytes, cudaMemcpyDeviceToHost, m.stream));
-    }
-    // the status words of the bounded waits travel with the result: one synchronisation per step, not one per word
+// Waits for the step and reports the bounded waits inside it: their status words travel with the result, one synchronisation per
+// step, not one per word.
+static int finish_step(Model &m) {
     int *hs = m.h_status;
     hs[0] = hs[1] = 0;
     if (m.gemm_ws) MYNN_CUDA_OK(cudaMemcpyAsync(&hs[0], m.gemm_ws, sizeof(int), cudaMemcpyDeviceToHost, m.stream));
@@ -569,6 +530,21 @@ static int copy_result_to_host(Model &m, void *dst) {
     return MYNN_OK;
 }
 
+// tp > 1 logits arrive as [rank][batch][vocab/tp]; reorder on the host side of the copy.
+static int copy_result_to_host(Model &m, void *dst) {
+    size_t bytes;
+    const void *src = result_ptr(m, &bytes);
+    if (m.c.output_mode == 0 && m.c.tp_world > 1) {
+        const size_t row = (size_t)m.vocab_l * dtype_size(m.c.dtype);
+        for (int r = 0; r < m.c.tp_world; r++)
+            MYNN_CUDA_OK(cudaMemcpy2DAsync((char *)dst + r * row, row * m.c.tp_world, (const char *)src + (size_t)r * m.c.batch * row,
+                                           row, row, m.c.batch, cudaMemcpyDeviceToHost, m.stream));
+    } else {
+        MYNN_CUDA_OK(cudaMemcpyAsync(dst, src, bytes, cudaMemcpyDeviceToHost, m.stream));
+    }
+    return finish_step(m);
+}
+
 static int model_run(Model &m, void **output, void **input) {
     if (!output || !input || !output[0] || !input[0] || !input[1] || !input[2] || !input[3])
         return fail(MYNN_E_ARG, "model: null input/output pointer");
@@ -577,6 +553,7 @@ static int model_run(Model &m, void **output, void **input) {
     if (past < 0 || past >= m.c.max_seq_len || active < 0 || active > m.c.max_seq_len)
         return fail(MYNN_E_ARG, "model: past_len %lld / active_seq_kv %lld outside the %d-row cache", (long long)past,
                     (long long)active, m.c.max_seq_len);
+    if (m.blocks) RC(block_admit(m, (int)past, 1));
     cudaStream_t st = m.stream;
     // one pinned block, one copy: {past, active, position, ids}
     ((int32_t *)m.h_in)[0] = (int32_t)past;
@@ -613,6 +590,25 @@ extern "C" int mynn_b200_model_configure(const mynn_b200_model_config *cfg) {
         return fail(MYNN_E_ARG, "model_configure: sink %d + window %d exceed max_seq_len %d", c.stream_sink, c.stream_window, c.max_seq_len);
     g_cfg = c;
     g_cfg_set = true;
+    g_cfg_blocks = false;
+    return MYNN_OK;
+}
+
+extern "C" int mynn_b200_model_configure_blocks(const mynn_b200_block_model_config *cfg) {
+    RC(block_configure(cfg));
+    mynn_b200_model_config c = {};  // what the entry points need to know of a model
+    c.n_layers = cfg->n_layers;
+    c.hidden = cfg->hidden;
+    c.vocab = cfg->vocab;
+    c.max_seq_len = cfg->max_seq_len;
+    c.batch = cfg->batch;
+    c.dtype = cfg->dtype;
+    c.output_mode = cfg->output_mode;
+    c.tp_world = 1;
+    c.use_graph = cfg->use_graph;
+    c.max_prefill = cfg->max_prefill;
+    g_cfg = c;
+    g_cfg_set = g_cfg_blocks = true;
     return MYNN_OK;
 }
 
@@ -643,6 +639,7 @@ extern "C" void model_destroy(void *state) {
     for (int r = 0; r < m->tp.world; r++)
         if (m->tp_attached && r != m->tp.rank && m->tp.blocks[r]) cudaIpcCloseMemHandle(m->tp.blocks[r]);
     if (m->tp_block) cudaFree(m->tp_block);
+    if (m->blocks) block_destroy(*m);
     delete m;
 }
 
@@ -653,6 +650,7 @@ extern "C" int mynn_b200_model_step_device(void *state, void *stream, const int6
     Model &m = *(Model *)state;
     if (m.c.stream_window > 0) return fail(MYNN_E_STATE, "model_step_device: this model has a streaming cache; step it with mynn_b200_model_stream");
     if (past_len < 0 || past_len >= m.c.max_seq_len) return fail(MYNN_E_ARG, "model_step_device: past_len %d outside the cache", past_len);
+    if (m.blocks) RC(block_admit(m, past_len, 1));
     cudaStream_t st = stream ? (cudaStream_t)stream : m.stream;
     // The 16-byte header is passed by value through a pageable copy (staged by the runtime before it returns).
     struct { int32_t past, active; int64_t pos; } hdr = {past_len, past_len + 1, (int64_t)past_len};
@@ -667,17 +665,13 @@ extern "C" int mynn_b200_model_step_device(void *state, void *stream, const int6
     return MYNN_OK;
 }
 
-// Prefill of T tokens per sequence starting at cache row past_len (the engine's prefill graph,
-// crates/llm/src/session.rs:426-480, without the padding rows): ids_host int64 [batch, T]; out_host receives the
-// logits / token ids of the last position, as model() does.  T <= max_prefill.
-extern "C" int mynn_b200_model_prefill(void *state, const int64_t *ids_host, int T, int past_len, void *out_host) {
-    if (!state) return fail(MYNN_E_STATE, "model_prefill: null state");
-    Model &m = *(Model *)state;
-    if (m.c.stream_window > 0) return fail(MYNN_E_STATE, "model_prefill: this model has a streaming cache; step it with mynn_b200_model_stream");
+// The inputs of a prefill chunk on the device.
+static int prefill_inputs(Model &m, const int64_t *ids_host, int T, int past_len, const char *what) {
+    if (m.c.stream_window > 0) return fail(MYNN_E_STATE, "%s: this model has a streaming cache; step it with mynn_b200_model_stream", what);
     const int cap = m.c.max_prefill > 0 ? m.c.max_prefill : 1;
-    if (T <= 0 || T > cap) return fail(MYNN_E_ARG, "model_prefill: %d tokens, capacity %d", T, cap);
-    if (past_len < 0 || past_len + T > m.c.max_seq_len) return fail(MYNN_E_ARG, "model_prefill: rows [%d, %d) outside the %d-row cache", past_len, past_len + T, m.c.max_seq_len);
-    if (!ids_host || !out_host) return fail(MYNN_E_ARG, "model_prefill: null pointer");
+    if (T <= 0 || T > cap) return fail(MYNN_E_ARG, "%s: %d tokens, capacity %d", what, T, cap);
+    if (past_len < 0 || past_len + T > m.c.max_seq_len) return fail(MYNN_E_ARG, "%s: rows [%d, %d) outside the %d-row cache", what, past_len, past_len + T, m.c.max_seq_len);
+    if (m.blocks) RC(block_admit(m, past_len, T));
     cudaStream_t st = m.stream;
     std::vector<int64_t> pos(T);
     for (int i = 0; i < T; i++) pos[i] = past_len + i;
@@ -686,8 +680,40 @@ extern "C" int mynn_b200_model_prefill(void *state, const int64_t *ids_host, int
     MYNN_CUDA_OK(cudaMemcpyAsync(m.pos_dev, pos.data(), (size_t)T * 8, cudaMemcpyHostToDevice, st));
     MYNN_CUDA_OK(cudaMemcpyAsync(m.past_dev, &hdr, 16, cudaMemcpyHostToDevice, st));
     MYNN_CUDA_OK(cudaStreamSynchronize(st));  // the sources above are short-lived host memory
-    RC(enqueue_forward(m, st, T));
+    return MYNN_OK;
+}
+
+// Prefill of T tokens per sequence starting at cache row past_len (the engine's prefill graph,
+// crates/llm/src/session.rs:426-480, without the padding rows): ids_host int64 [batch, T]; out_host receives the
+// logits / token ids of the last position, as model() does.  T <= max_prefill.
+extern "C" int mynn_b200_model_prefill(void *state, const int64_t *ids_host, int T, int past_len, void *out_host) {
+    if (!state) return fail(MYNN_E_STATE, "model_prefill: null state");
+    Model &m = *(Model *)state;
+    if (!ids_host || !out_host) return fail(MYNN_E_ARG, "model_prefill: null pointer");
+    RC(prefill_inputs(m, ids_host, T, past_len, "model_prefill"));
+    RC(enqueue_forward(m, m.stream, T));
     return copy_result_to_host(m, out_host);
+}
+
+// The same chunk, but the logits of chosen rows of [batch * T] are returned (none: the chunk only enters the cache).
+extern "C" int mynn_b200_model_prefill_rows(void *state, const int64_t *ids_host, int T, int past_len, const int32_t *rows_host, int n_rows,
+                                            void *out_host) {
+    if (!state) return fail(MYNN_E_STATE, "model_prefill_rows: null state");
+    Model &m = *(Model *)state;
+    if (!ids_host || n_rows < 0 || (n_rows > 0 && (!rows_host || !out_host))) return fail(MYNN_E_ARG, "model_prefill_rows: null pointer");
+    if (m.c.output_mode != 0 || m.c.tp_world > 1) return fail(MYNN_E_UNSUPPORTED, "model_prefill_rows: needs a model that returns logits, not tensor parallel");
+    if (n_rows > m.head_capacity) return fail(MYNN_E_ARG, "model_prefill_rows: %d rows, capacity %d", n_rows, m.head_capacity);
+    for (int i = 0; i < n_rows; i++)
+        if (rows_host[i] < 0 || rows_host[i] >= m.c.batch * T) return fail(MYNN_E_ARG, "model_prefill_rows: row %d outside [0, %d)", rows_host[i], m.c.batch * T);
+    RC(prefill_inputs(m, ids_host, T, past_len, "model_prefill_rows"));
+    if (n_rows > 0) {
+        MYNN_CUDA_OK(cudaMemcpyAsync(m.rows_dev, rows_host, (size_t)n_rows * 4, cudaMemcpyHostToDevice, m.stream));
+        MYNN_CUDA_OK(cudaStreamSynchronize(m.stream));  // the caller's memory
+    }
+    RC(enqueue_forward(m, m.stream, T, n_rows > 0 ? n_rows : -1));
+    if (n_rows > 0)
+        MYNN_CUDA_OK(cudaMemcpyAsync(out_host, m.logits, (size_t)n_rows * m.c.vocab * dtype_size(m.logits_dtype), cudaMemcpyDeviceToHost, m.stream));
+    return finish_step(m);
 }
 
 // Streaming step.  Token P of the stream lives in slot P (P < sink) or sink + (P - sink) % window.  After the append

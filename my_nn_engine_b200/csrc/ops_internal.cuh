@@ -98,6 +98,9 @@ int launch_argmax_merge(cudaStream_t st, int32_t *out_idx, const float *pairs /*
 int launch_argmax_two_stage(cudaStream_t st, int dtype, int32_t *out_idx, float *pairs /*[chunks][rows][2]*/, const void *logits,
                             int rows, int V, int chunks);
 
+// out row i = x row rows_dev[i], rows of row_bytes (a multiple of 4).
+int launch_gather_rows(cudaStream_t st, void *out, const void *x, const int32_t *rows_dev, int rows, size_t row_bytes);
+
 // ids[i] = tok[i]: feeds the greedy tokens back as the next step's input ids without leaving the device.
 int launch_tok_feedback(cudaStream_t st, int64_t *ids, const int32_t *tok, int n);
 

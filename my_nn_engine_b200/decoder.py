@@ -65,7 +65,114 @@ def _shard_heads(t, n_heads, rank, world):
     return t[h0 * per:h1 * per]
 
 
-class DecoderModel:
+MAX_HEAD_ROWS = 64  # logits rows per prefill chunk (mynn_b200_model_prefill_rows)
+
+
+class DeviceModel:
+    """A model resident on the current CUDA device behind the library's model entry points: what every model family shares.
+
+    A subclass lays out its weights and state buffers and calls ``_open`` with its configuration; steps, prefill chunks and
+    their host staging are the same for all."""
+
+    def _open(self, configure, config, init, states, logits_dtype):
+        """configure + model_init, then the pinned host staging."""
+        self.lib = ffi.lib()
+        ffi.check(configure(ctypes.byref(config)))
+        self._init_arr = (ctypes.c_void_p * len(init))(*init)
+        self._state_arr = (ctypes.c_void_p * len(states))(*states)
+        with torch.cuda.device(self.device):
+            self.state = self.lib.model_init(self._init_arr, self._state_arr)
+        ffi.check(self.lib.mynn_b200_model_status())
+        if not self.state:
+            raise RuntimeError("model_init returned no state")
+        # host staging in pinned memory, as the engine's alloc_pinned buffers
+        batch = self.batch
+        self._ids = torch.zeros(batch, dtype=torch.int64).pin_memory()
+        self._scalars = torch.zeros(3, dtype=torch.int64).pin_memory()  # position_id, past_len, active_seq_kv
+        n_out = batch if self.output == "ids" else batch * self.vocab
+        self._logits_dtype = logits_dtype
+        self._out = torch.zeros(n_out, dtype=torch.int32 if self.output == "ids" else logits_dtype).pin_memory()
+        sp = self._scalars.data_ptr()
+        self._in_arr = (ctypes.c_void_p * 4)(self._ids.data_ptr(), sp, sp + 8, sp + 16)
+        self._out_arr = (ctypes.c_void_p * 1)(self._out.data_ptr())
+        self.h2d_bytes_per_step = 16 + 8 * batch
+        self.d2h_bytes_per_step = self._out.numel() * self._out.element_size()
+
+    def step(self, tokens, past_len: int, active_seq_kv: int | None = None):
+        """One decode step through ``model(state, outputs, inputs)`` with HOST buffers: inputs are
+        input_ids [batch,1], position_id [1] = past_len, past_len, active_seq_kv = past_len + 1
+        (crates/llm/src/session.rs:508-537).  Returns a pinned host tensor: logits [batch, vocab] or ids [batch]."""
+        self._ids.copy_(torch.as_tensor(tokens, dtype=torch.int64).reshape(self.batch))
+        self._scalars[0] = past_len
+        self._scalars[1] = past_len
+        self._scalars[2] = past_len + 1 if active_seq_kv is None else active_seq_kv
+        self.lib.model(self.state, self._out_arr, self._in_arr)
+        ffi.check(self.lib.mynn_b200_model_status())
+        return self._out if self.output == "ids" else self._out.view(self.batch, self.vocab)
+
+    def prefill(self, tokens, past_len: int):
+        """Prefill T tokens per sequence at cache rows [past_len, past_len+T); returns what step() returns for the
+        last position."""
+        ids = torch.as_tensor(tokens, dtype=torch.int64).reshape(self.batch, -1).contiguous()
+        ffi.check(self.lib.mynn_b200_model_prefill(self.state, ids.data_ptr(), ids.shape[1], past_len, self._out.data_ptr()))
+        return self._out if self.output == "ids" else self._out.view(self.batch, self.vocab)
+
+    def step_device(self, ids_dev, past_len: int, out_dev=None, stream=None):
+        """Device-resident step: ids int64 CUDA tensor [batch] (or None to reuse the resident ids); no host sync."""
+        st = stream if stream is not None else torch.cuda.current_stream().cuda_stream
+        ffi.check(self.lib.mynn_b200_model_step_device(self.state, st, None if ids_dev is None else ids_dev.data_ptr(),
+                                                       past_len, None if out_dev is None else out_dev.data_ptr()))
+
+    def prefill_rows(self, tokens, past_len: int, rows):
+        """The chunk of prefill() with the logits of chosen tokens: ``rows`` are indices b * T + t into the chunk; returns a host
+        tensor [len(rows), vocab]."""
+        ids = torch.as_tensor(tokens, dtype=torch.int64).reshape(self.batch, -1).contiguous()
+        sel = torch.as_tensor(list(rows), dtype=torch.int32)
+        out = torch.empty(len(sel), self.vocab, dtype=self._logits_dtype)
+        ffi.check(self.lib.mynn_b200_model_prefill_rows(self.state, ids.data_ptr(), ids.shape[1], past_len, sel.data_ptr(), len(sel),
+                                                        out.data_ptr()))
+        return out
+
+    def feed(self, tokens, past_len: int, want=()):
+        """Run the next ``tokens`` of the one sequence (batch 1) from cache row past_len on, in prefill chunks or, where a chunk
+        is one token, as a decode step; returns the f32 logits [len(want), vocab] at the places ``want`` among these tokens."""
+        if self.batch != 1 or self.output != "logits":
+            raise ValueError("feed() needs a batch-1 model that returns logits")
+        tokens, want = [int(t) for t in tokens], [int(w) for w in want]
+        if any(not 0 <= w < len(tokens) for w in want):
+            raise ValueError("feed(): a wanted place lies outside the tokens given")
+        out = torch.empty(len(want), self.vocab, dtype=torch.float32)
+        cap, asked, pos = max(self.max_prefill, 1), set(want), 0
+        while pos < len(tokens):
+            size = min(cap, len(tokens) - pos)
+            here = [w for w in sorted(asked) if pos <= w < pos + size]
+            if len(here) > MAX_HEAD_ROWS:  # the chunk ends in front of the first place that has no room
+                size = here[MAX_HEAD_ROWS] - pos
+                here = here[:MAX_HEAD_ROWS]
+            if size == 1:
+                got = self.step([tokens[pos]], past_len + pos)
+            else:
+                got = self.prefill_rows([tokens[pos:pos + size]], past_len + pos, [w - pos for w in here])
+            for i, w in enumerate(here):
+                for j, v in enumerate(want):
+                    if v == w:
+                        out[j] = got[i].float()
+            pos += size
+        return out
+
+    def close(self):
+        if getattr(self, "state", None):
+            self.lib.model_destroy(self.state)
+            self.state = None
+
+    def __del__(self):
+        try:
+            self.close()
+        except Exception:
+            pass
+
+
+class DecoderModel(DeviceModel):
     """One tensor-parallel rank of a Llama-family decoder resident on the current CUDA device.
 
     cfg: HF config dict.  state: HF-named tensors with int8 weights and ``<name>.scale`` vectors (the engine's
@@ -174,14 +281,8 @@ class DecoderModel:
                             kv_int8=int(kv_int8), stream_sink=streaming[0] if streaming else 0,
                             stream_window=streaming[1] if streaming else 0,
                             rms_eps=cfg["rms_norm_eps"])
-        ffi.check(self.lib.mynn_b200_model_configure(ctypes.byref(c)))
-        self._init_arr = (ctypes.c_void_p * len(init))(*init)
-        self._state_arr = (ctypes.c_void_p * len(states))(*states)
-        with torch.cuda.device(dev):
-            self.state = self.lib.model_init(self._init_arr, self._state_arr)
-        ffi.check(self.lib.mynn_b200_model_status())
-        if not self.state:
-            raise RuntimeError("model_init returned no state")
+        self.max_prefill = max_prefill
+        self._open(self.lib.mynn_b200_model_configure, c, init, states, td)
         self.tp_fused = False
         if G > 1 and tp_fused and tensor_gemm and batch <= 32 and h % 16 == 0:
             # hand every rank's partial-sum block to every other rank (64-byte IPC handles over torch.distributed)
@@ -194,17 +295,6 @@ class DecoderModel:
             ffi.check(self.lib.mynn_b200_model_tp_attach(self.state, blob))
             self.tp_fused = True
 
-        # host staging in pinned memory, as the engine's alloc_pinned buffers
-        self._ids = torch.zeros(batch, dtype=torch.int64).pin_memory()
-        self._scalars = torch.zeros(3, dtype=torch.int64).pin_memory()  # position_id, past_len, active_seq_kv
-        n_out = batch if output == "ids" else batch * self.vocab
-        self._out = torch.zeros(n_out, dtype=torch.int32 if output == "ids" else td).pin_memory()
-        sp = self._scalars.data_ptr()
-        self._in_arr = (ctypes.c_void_p * 4)(self._ids.data_ptr(), sp, sp + 8, sp + 16)
-        self._out_arr = (ctypes.c_void_p * 1)(self._out.data_ptr())
-        self.h2d_bytes_per_step = 16 + 8 * batch
-        self.d2h_bytes_per_step = self._out.numel() * self._out.element_size()
-
     # ---- the engine's Session::run for the decode graph ----
     @classmethod
     def from_pretrained(cls, model_dir: str, **kwargs):
@@ -214,25 +304,6 @@ class DecoderModel:
         cfg, state = load_model_dir(model_dir)
         return cls(cfg, state, **kwargs)
 
-    def step(self, tokens, past_len: int, active_seq_kv: int | None = None):
-        """One decode step through ``model(state, outputs, inputs)`` with HOST buffers: inputs are
-        input_ids [batch,1], position_id [1] = past_len, past_len, active_seq_kv = past_len + 1
-        (crates/llm/src/session.rs:508-537).  Returns a pinned host tensor: logits [batch, vocab] or ids [batch]."""
-        self._ids.copy_(torch.as_tensor(tokens, dtype=torch.int64).reshape(self.batch))
-        self._scalars[0] = past_len
-        self._scalars[1] = past_len
-        self._scalars[2] = past_len + 1 if active_seq_kv is None else active_seq_kv
-        self.lib.model(self.state, self._out_arr, self._in_arr)
-        ffi.check(self.lib.mynn_b200_model_status())
-        return self._out if self.output == "ids" else self._out.view(self.batch, self.vocab)
-
-    def prefill(self, tokens, past_len: int):
-        """Prefill T tokens per sequence at cache rows [past_len, past_len+T); returns what step() returns for the
-        last position."""
-        ids = torch.as_tensor(tokens, dtype=torch.int64).reshape(self.batch, -1).contiguous()
-        ffi.check(self.lib.mynn_b200_model_prefill(self.state, ids.data_ptr(), ids.shape[1], past_len, self._out.data_ptr()))
-        return self._out if self.output == "ids" else self._out.view(self.batch, self.vocab)
-
     def stream(self, tokens, stream_pos: int):
         """Streaming-cache step: tokens [batch] (a decode step) or [batch, T] (a prefill chunk that must not evict) at
         absolute stream positions stream_pos..; returns what step() returns for the last position."""
@@ -240,26 +311,9 @@ class DecoderModel:
         ffi.check(self.lib.mynn_b200_model_stream(self.state, ids.data_ptr(), ids.shape[1], int(stream_pos), self._out.data_ptr()))
         return self._out if self.output == "ids" else self._out.view(self.batch, self.vocab)
 
-    def step_device(self, ids_dev, past_len: int, out_dev=None, stream=None):
-        """Device-resident step: ids int64 CUDA tensor [batch] (or None to reuse the resident ids); no host sync."""
-        st = stream if stream is not None else torch.cuda.current_stream().cuda_stream
-        ffi.check(self.lib.mynn_b200_model_step_device(self.state, st, None if ids_dev is None else ids_dev.data_ptr(),
-                                                       past_len, None if out_dev is None else out_dev.data_ptr()))
-
     def reset_cache(self):
         for t in self.k_cache + self.v_cache + self.k_scale + self.v_scale:
             t.zero_()
 
     def weight_bytes(self) -> int:
         return sum(t.numel() for t in self._keep if t.dtype == torch.int8)
-
-    def close(self):
-        if getattr(self, "state", None):
-            self.lib.model_destroy(self.state)
-            self.state = None
-
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass

@@ -32,6 +32,21 @@ class ModelConfig(ctypes.Structure):
                                        "use_graph", "max_prefill", "use_tensor_gemm", "stream_sink", "stream_window", "kv_int8")] + [("rms_eps", c_float)]
 
 
+class Block(ctypes.Structure):
+    """Mirror of ``mynn_b200_block``: one layer of a block decoder."""
+
+    _fields_ = [(n, c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "conv_taps", "rot_dims", "window", "cache_rows", "history_rows",
+                                       "experts", "expert_ff", "top", "groups", "groups_keep")] + [("attn_scale", c_float), ("softcap", c_float)]
+
+
+class BlockModelConfig(ctypes.Structure):
+    """Mirror of ``mynn_b200_block_model_config``."""
+
+    _fields_ = [(n, c_int32) for n in ("n_layers", "hidden", "vocab", "max_seq_len", "batch", "dtype", "output_mode", "use_graph", "max_prefill",
+                                       "max_rewind", "loop_start", "loop_stop", "loop_times")] + \
+               [(n, c_float) for n in ("embed_scale", "residual_mult", "norm_eps")] + [("layers", POINTER(Block))]
+
+
 class TpGroup(ctypes.Structure):
     """Mirror of ``mynn_b200_tp_group`` (include/mynn_b200.h)."""
 
@@ -87,6 +102,16 @@ SIGNATURES = {
     "mynn_b200_model_step_device": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_void_p]),
     "mynn_b200_model_prefill": (c_int, [c_void_p, c_void_p, c_int, c_int, c_void_p]),
     "mynn_b200_model_stream": (c_int, [c_void_p, c_void_p, c_int, c_int64, c_void_p]),
+    "mynn_b200_model_prefill_rows": (c_int, [c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p]),
+    "mynn_b200_model_configure_blocks": (c_int, [POINTER(BlockModelConfig)]),
+    "mynn_b200_layer_norm": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int]),
+    "mynn_b200_residual_layer_norm": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int]),
+    "mynn_b200_short_conv_append": (c_int, [c_void_p] * 9 + [c_int] * 10 + [c_void_p, c_int]),
+    "mynn_b200_window_attention": (c_int, [c_void_p] * 5 + [c_float, c_float] + [c_int] * 9 + [c_void_p, c_int, c_void_p, c_size_t, c_int]),
+    "mynn_b200_moe_workspace_bytes": (c_size_t, [c_int, c_int, c_int]),
+    "mynn_b200_moe_route": (c_int, [c_void_p, c_void_p, c_size_t, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int]),
+    "mynn_b200_dense_matmul": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "mynn_b200_moe_matmul": (c_int, [c_void_p] * 6 + [c_int] * 9 + [c_void_p]),
     "mynn_b200_model_tp_export": (c_int, [c_void_p, c_void_p]),
     "mynn_b200_model_tp_attach": (c_int, [c_void_p, c_void_p]),
     "mynn_b200_attention_decode_splits": (c_int, [c_int, c_int, c_int, c_int]),

@@ -48,6 +48,7 @@ class LlmSession:
         self.prefill_len = prefill_len if prefill is not None else None
         self.tokenizer = tokenizer
         self._past_len = 0
+        self._feed = None
         self.streaming = None  # (sink, window) when bound to a streaming-cache model: the stream has no length limit
 
     @classmethod
@@ -87,6 +88,25 @@ class LlmSession:
             return pick(model.prefill([list(ids)], past_len))
 
         return cls(step, model.max_seq_len, eos_token_id, prefill if prefill_len else None, prefill_len, tokenizer)
+
+    @classmethod
+    def for_model(cls, model, eos_token_id: int, prefill_len: Optional[int] = None, tokenizer=None):
+        """Bind to any batch-1 model of the registry (a streaming-cache model steps by stream position)."""
+        make = cls.for_llama_streaming if getattr(model, "streaming", None) else cls.for_llama
+        self = make(model, eos_token_id, prefill_len, tokenizer)
+        self._feed = getattr(model, "feed", None)
+        return self
+
+    def feed(self, tokens: Sequence[int], want: Sequence[int] = ()):
+        """Append given tokens to the sequence without picking any: prefill chunks and decode steps at the current past_len.
+        Returns the logits at the places ``want`` among them (a model bound with ``for_model`` that returns logits)."""
+        if self._feed is None or self.streaming:
+            raise ValueError("feed() needs a model bound with for_model() and a plain cache")
+        if self.max_seq_len < self._past_len + len(tokens):
+            raise PromptTooLong(self._past_len + len(tokens), self.max_seq_len, self._past_len)
+        out = self._feed(tokens, self._past_len, want)
+        self._past_len += len(tokens)
+        return out
 
     def past_len(self) -> int:
         return self._past_len
