@@ -2,7 +2,7 @@
 batch 32, 2048-token context, greedy decode — tokens per second of the whole job.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
-    python bench.py --case {gemv|gemm|attention|prefill_gemm|prefill_attention|prefill_model|w8a8|suite} [...]
+    python bench.py --case {gemv|gemm|attention|prefill_gemm|prefill_attention|prefill_model|w8a8|suite|block|block_kernels} [...]
 
 Default case ("step").  A step is one decode step of the whole batch (32 new tokens).  Weights are random-init (N(0, 0.02),
 quantised with the engine's quantizer), the 2048-token context is synthetic KV (N(0,1) * 0.5, one seed for the whole cache,
@@ -22,6 +22,8 @@ cannot be built here) with all host threads.
 
 The other cases time single kernels of the path the way the step's kernels are fed: every launch reads a different copy of
 its weights / KV (copies x size > L2), the launches are replayed from one CUDA graph, CUDA events on the launching stream.
+block: prefill and decode throughput of Vebisun-shaped models with layers like those of real ones, beside the int8 Llama graph at
+equal width, heads, depth and feed-forward width per token; block_kernels: their kernels one by one against the roofline.
 Algorithmic bytes: GEMM  N*K + N*sizeof(scale) + M*K*sizeof(act) + M*N*sizeof(out);  attention  2*B*Hkv*L*D*2 + Q + out.
 """
 from __future__ import annotations
@@ -710,11 +712,198 @@ def case_w8a8(m, n, k, dtype="bf16", copies=None):
             "frac_of_%s_hbm_peak" % kind: alg / us / 1e3 / hbm, "algorithmic_bytes": alg}
 
 
+# --------------------------------------------------------------------------------------------------------
+# block decoders (Vebisun): layers like those of real models, random weights, beside the int8 Llama graph at equal size
+# --------------------------------------------------------------------------------------------------------
+# (width, heads, kv heads, head size, window, experts, top, expert ff, groups, kept groups, layers, vocabulary)
+BLOCK_ARCHS = {
+    "small-experts": dict(width=2048, heads=32, kv=8, dim=128, window=1024, experts=64, top=8, ff=1024, groups=8, keep=4, layers=8, vocab=32000),
+    "large-experts": dict(width=4096, heads=32, kv=8, dim=128, window=4096, experts=8, top=2, ff=7168, groups=4, keep=2, layers=4, vocab=32000),
+}
+
+
+def block_model(a, batch, max_seq, max_prefill, output="ids", loop=None, max_rewind=256):
+    """A Vebisun-shaped block decoder of one of BLOCK_ARCHS with random bf16 weights made on the device."""
+    import torch
+
+    from my_nn_engine_b200.block_decoder import BlockDecoder, BlockLayer, BlockModelSpec, Rotary, RotaryScaling
+    g = torch.Generator(device="cuda").manual_seed(0)
+
+    def mat(*shape):
+        return torch.empty(*shape, device="cuda", dtype=torch.bfloat16).normal_(0.0, 0.02, generator=g)
+
+    def norm():
+        return torch.ones(a["width"], device="cuda"), torch.zeros(a["width"], device="cuda")
+
+    W = a["width"]
+    L = BlockLayer(heads=a["heads"], kv_heads=a["kv"], dim=a["dim"], vdim=a["dim"], scale=a["dim"] ** -0.5, softcap=30.0, window=a["window"], conv_taps=4,
+                   rotary=Rotary(5e5, a["dim"] // 2, RotaryScaling(8.0, 1.0, 4.0, 8192.0)), experts=a["experts"], expert_ff=a["ff"], top=a["top"],
+                   groups=a["groups"], groups_keep=a["keep"])
+    spec = BlockModelSpec(hidden=W, vocab=a["vocab"], layers=[L] * a["layers"], norm_eps=1e-5, embed_scale=1.0, residual_mult=0.5, loop=loop)
+    weights = {"embed": mat(a["vocab"], W), "head": mat(a["vocab"], W), "final_norm": norm(), "layers": [
+        {"norm1": norm(), "norm1b": norm(), "norm2": norm(), "norm2b": norm(), "qkv": mat(L.channels, W), "conv": mat(L.channels, 4), "o": mat(W, L.heads * L.vdim),
+         "router": mat(L.experts, W), "gate_up": mat(L.experts, 2 * L.expert_ff, W), "down": mat(L.experts, W, L.expert_ff)} for _ in range(a["layers"])]}
+    return BlockDecoder(spec, weights, dtype="bf16", max_seq_len=max_seq, batch=batch, output=output, max_prefill=max_prefill, max_rewind=max_rewind)
+
+
+def llama_beside(a, batch, max_seq, max_prefill):
+    """The int8 Llama graph with the same width, heads, depth and vocabulary; its feed-forward is as wide as the experts a token uses."""
+    from my_nn_engine_b200.decoder import DecoderModel
+    from my_nn_engine_b200.quantize import random_llama_state
+    cfg = dict(hidden_size=a["width"], num_hidden_layers=a["layers"], num_attention_heads=a["heads"], num_key_value_heads=a["kv"], head_dim=a["dim"],
+               intermediate_size=a["ff"] * a["top"], vocab_size=a["vocab"], rms_norm_eps=1e-5, rope_theta=500000.0)
+    return DecoderModel(cfg, random_llama_state(cfg, seed=0, device="cuda"), dtype="bf16", max_seq_len=max_seq, batch=batch, output="ids", max_prefill=max_prefill)
+
+
+def _model_throughput(model, vocab, batch, context, steps=64, chunk=2048):
+    """(prefill tokens/s of a fresh prompt of ``context`` tokens per sequence, decode ms per step behind it).  Wall clock around the
+    host call for the prefill (best of 3), CUDA events around device-resident steps for the decode."""
+    import torch
+    g = torch.Generator().manual_seed(1)
+    prompt = torch.randint(0, vocab, (batch, context), generator=g)
+    chunk = min(chunk, context)
+    best = 1e30
+    for _ in range(4):
+        torch.cuda.synchronize()
+        t0 = time.perf_counter()
+        for p in range(0, context, chunk):
+            model.prefill(prompt[:, p:p + chunk], p)
+        torch.cuda.synchronize()
+        best = min(best, time.perf_counter() - t0)
+    stream = torch.cuda.Stream()
+    ids = prompt[:, -1].contiguous().cuda()
+    torch.cuda.synchronize()
+    with torch.cuda.stream(stream):
+        for i in range(8):
+            model.step_device(ids if i == 0 else None, context + i)
+        times = []
+        for _ in range(3):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(stream)
+            for i in range(steps):
+                model.step_device(None, context + 8 + i)
+            e1.record(stream)
+            torch.cuda.synchronize()
+            times.append(e0.elapsed_time(e1) / steps)
+    return batch * context / best, sorted(times)[1]
+
+
+def case_block(name, batch, context=2048):
+    """Prefill and decode throughput of one block architecture and of the Llama graph beside it."""
+    import torch
+    a = BLOCK_ARCHS[name]
+    chunk = max(64, 2048 // batch)
+    out = {"case": "block", "arch": name, **a, "batch": batch, "context": context, "chunk": chunk, "data": "synthetic"}
+    for key, make in (("vebisun_bf16", block_model), ("llama_int8", llama_beside)):
+        m = make(a, batch, context + 128, chunk)
+        l0 = m.lib.mynn_b200_launch_count()
+        tps, ms = _model_throughput(m, a["vocab"], batch, context, chunk=chunk)
+        out[key] = {"prefill_tok_per_s": tps, "decode_ms_per_step": ms, "decode_tok_per_s": batch * 1e3 / ms, "weight_bytes": m.weight_bytes(),
+                    "kernels_launched": m.lib.mynn_b200_launch_count() - l0}
+        m.close()
+        del m
+        torch.cuda.empty_cache()
+    return out
+
+
+def case_block_kernels(name, batch, context=2048):
+    """The kernels of one block layer at a decode step of ``batch`` rows (batch > 32: at a prefill chunk of that many tokens) against
+    their rooflines, each next to the like kernel of the Llama graph at the same shape."""
+    import torch
+
+    from my_nn_engine_b200 import ops
+    a, M = BLOCK_ARCHS[name], batch
+    hbm, tf, kind = measured_peaks()
+    W, H, G, D, E, top, ff = (a[k] for k in ("width", "heads", "kv", "dim", "experts", "top", "ff"))
+    C = (H + 2 * G) * D
+    prefill = M > 32
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+
+    def rnd(*shape):
+        return torch.empty(*shape, device="cuda", dtype=torch.bfloat16).normal_(0.0, 0.05)
+
+    def figure(what, us, nbytes, flops, **more):
+        r = {"case": "block_kernels", "arch": name, "rows": M, "kernel": what, "us": us, **more}
+        r.update({"bound": "tensor", "TFLOPs": flops / us / 1e6, "frac_of_%s" % kind: flops / us / 1e6 / tf} if prefill else
+                 {"bound": "hbm", "GBps": nbytes / us / 1e3, "frac_of_%s" % kind: nbytes / us / 1e3 / hbm})
+        return r
+
+    def copies(nbytes):
+        return max(3, int(400e6 // nbytes) + 1)
+
+    for what, N, K in (("qkv", C, W), ("o", W, H * D), ("head", a["vocab"], W)):
+        if prefill and what == "head":
+            continue
+        act = rnd(M, K)
+        ws = [rnd(N, K) for _ in range(copies(2 * N * K))]
+        out = torch.empty(M, N, device="cuda", dtype=torch.bfloat16)
+        us = _time_launches([(lambda w=w: ops.dense_matmul(act, w, out=out, status=status)) for w in ws])
+        yield figure(f"dense_matmul {what} {N}x{K}", us, 2 * (N * K + M * K + M * N), 2.0 * M * N * K)
+        del ws
+        like = case_gemm(M, N, K)
+        yield {**like, "case": "block_kernels", "arch": name, "like": f"dense_matmul {what}"}
+    # experts: the chosen blocks are read once; the routing (and the distribution of tokens) is random
+    logits = torch.randn(M, E, device="cuda")
+    r = ops.MoeRouting(logits, top, a["groups"], a["keep"])
+    used = int(torch.unique(r.chosen).numel())
+    h = rnd(M, W)
+    n_cp = max(2, int(600e6 // (used * 6 * W * ff)) + 1)
+    gus, dns = [rnd(E, 2 * ff, W) for _ in range(n_cp)], [rnd(E, W, ff) for _ in range(n_cp)]
+    hid = r.matmul(h, gus[0], gather=True, glu=True)
+    us = _time_launches([(lambda w=w: r.matmul(h, w, gather=True, glu=True)) for w in gus])
+    yield figure(f"experts gate/up ({used} of {E} used)", us, 2 * (used * 2 * ff * W + M * W + M * top * ff), 4.0 * M * top * ff * W)
+    us = _time_launches([(lambda w=w: r.matmul(hid, w, gather=False)) for w in dns])
+    yield figure(f"experts down ({used} of {E} used)", us, 2 * (used * ff * W + M * top * (ff + W)), 2.0 * M * top * ff * W)
+    del gus, dns
+    if not prefill:  # the Llama graph's products of the same bytes
+        for what, N, K in (("gate/up", 2 * ff * top, W), ("down", W, ff * top)):
+            yield {**case_gemm(M, N, K), "case": "block_kernels", "arch": name, "like": "experts " + what}
+    us = _time_launches([lambda: ops.MoeRouting(logits, top, a["groups"], a["keep"])] * 8)
+    yield {"case": "block_kernels", "arch": name, "rows": M, "kernel": "route (with the workspace's zero fill and two copies)", "us": us}
+    # attention
+    if prefill:
+        S = M
+        rows = -(-(min(a["window"] - 1, context) + S) // 128) * 128
+        q, k, v = rnd(1, H, S, D), rnd(1, G, rows, D), rnd(1, G, rows, D)
+        seen = sum(min(i + 1, a["window"]) for i in range(S))
+        for cap in (30.0, 0.0):
+            us = _time_launches([lambda: ops.window_attention(q, k, v, D ** -0.5, S, a["window"], cap)] * 4)
+            yield figure(f"window attention, prefill {S} tokens, window {a['window']}, soft cap {cap}", us, 0, 4.0 * seen * D * H)
+        ops.attention_check()
+        yield {**case_prefill_attention(1, H, G, D, S), "case": "block_kernels", "arch": name, "like": "window attention"}
+    else:
+        n = min(a["window"], context)
+        rows = -(-(a["window"] + 256) // 128) * 128
+        kv = 2 * M * G * n * D * 2
+        ks, vs = [[rnd(M, G, rows, D) for _ in range(copies(kv // 2))] for _ in range(2)]
+        q = rnd(M, H, 1, D)
+        us = _time_launches([(lambda k=k, v=v: ops.window_attention(q, k, v, D ** -0.5, context, a["window"], 30.0)) for k, v in zip(ks, vs)])
+        ops.attention_check()
+        yield figure(f"window attention, decode, {n} rows seen", us, kv + 4 * q.numel(), 0)
+        del ks, vs
+        yield {**case_attention(M, H, G, D, n), "case": "block_kernels", "arch": name, "like": "window attention"}
+    # row kernels: bytes of x, the sublayer output and the normed row
+    x, sub = torch.randn(M, W, device="cuda"), rnd(M, W)
+    pn = (torch.ones(W, device="cuda"), torch.zeros(W, device="cuda"))
+    us = _time_launches([lambda: ops.residual_layer_norm(x, sub, pn, 0.5, 1e-5, norm=pn)] * 16)
+    yield {"case": "block_kernels", "arch": name, "rows": M, "kernel": "post norm + residual + norm", "us": us, "GBps": M * W * 12 / us / 1e3}
+    B, S = (1, M) if prefill else (M, 1)
+    proj, hist = rnd(B, S, C), rnd(B, 36, C)
+    kc, vc = rnd(B, G, -(-(a["window"] + S) // 128) * 128, D), rnd(B, G, -(-(a["window"] + S) // 128) * 128, D)
+    tab = torch.rand(max(context, S) + 1, D // 4, device="cuda")
+    conv, past = torch.rand(4, C, device="cuda"), torch.tensor([0 if prefill else context], dtype=torch.int32, device="cuda")
+    us = _time_launches([lambda: ops.short_conv_append(proj, past, kc, vc, H, conv, hist, tab, tab)] * 16)
+    yield {"case": "block_kernels", "arch": name, "rows": M, "kernel": "convolution + rotation + append", "us": us, "GBps": M * C * 4 / us / 1e3}
+    if int(status.item()):
+        raise RuntimeError(f"dense_matmul: a bounded wait ran out (status {int(status.item())})")
+
+
 def run_case(args):
     def emit(res):
         print(json.dumps(res), flush=True)
 
     c = args.case
+    args.b_given, args.m_given = args.b is not None, args.m is not None
     prefill = c in ("prefill_gemm", "w8a8")
     args.m = args.m or (2048 if prefill else 32)
     args.n = args.n or (14336 if prefill else 28672)
@@ -738,6 +927,15 @@ def run_case(args):
         emit(case_prefill_model(args.arch, args.b, args.len, args.chunk, args.layers, args.dtype, kv_int8=args.kv == "int8"))
     elif c == "decode_model":
         emit(case_decode_model(args.arch, args.b, dtype=args.dtype))
+    elif c == "block":
+        for name in ([args.block] if args.block else BLOCK_ARCHS):
+            for batch in ([args.b] if args.b_given else (1, 32)):
+                emit(case_block(name, batch, args.len))
+    elif c == "block_kernels":
+        for name in ([args.block] if args.block else BLOCK_ARCHS):
+            for rows in ([args.m] if args.m_given else (1, 32, 2048)):
+                for res in case_block_kernels(name, rows, args.len):
+                    emit(res)
     elif c == "w8a8":
         emit(case_w8a8(args.m, args.n, args.k, args.dtype, args.copies))
     elif c == "suite":
@@ -776,6 +974,7 @@ def main():
     ap.add_argument("--dtype", default="bf16")
     ap.add_argument("--kernel", default="tcgen05_i8", choices=["tcgen05_i8", "mma_sync"])
     ap.add_argument("--layout", default="nk", choices=["nk", "kn"])
+    ap.add_argument("--block", choices=sorted(BLOCK_ARCHS), help="one architecture of --case block / block_kernels (default: all)")
     ap.add_argument("--arch", default="llama3-8b", choices=["llama3-8b", "tinyllama"])
     ap.add_argument("--option", action="append", default=[], metavar="NAME=VALUE",
                     help="library option set before the run (mynn_b200_set_option), e.g. decode_ring=0, fuse_rope=0, ksplit=4")

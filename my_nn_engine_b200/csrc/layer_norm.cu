@@ -196,14 +196,17 @@ __global__ void __launch_bounds__(NV == 1 ? 256 : 1024) norm_step_kernel(const N
 template <typename T, int V>
 static int run_norm(cudaStream_t st, const NormStep &p, int rows) {
     const int groups = (p.W + V - 1) / V;
-    const int nv = groups <= 256 ? 1 : groups <= 2048 ? 2 : groups <= 4096 ? 4 : groups <= 8192 ? 8 : 0;
+    const int nv = groups <= 256 ? 1 : groups <= 2048 ? 2 : groups <= 4096 ? 4 : groups <= 8192 ? 8 : V == 1 && groups <= 32768 ? 32 : 0;
     if (!nv) return fail(MYNN_E_UNSUPPORTED, "layer_norm: rows of %d elements", p.W);
     const int threads = ((groups + nv - 1) / nv + 31) / 32 * 32;
     switch (nv) {
         case 1: norm_step_kernel<T, V, 1><<<rows, threads, 0, st>>>(p); break;
         case 2: norm_step_kernel<T, V, 2><<<rows, threads, 0, st>>>(p); break;
         case 4: norm_step_kernel<T, V, 4><<<rows, threads, 0, st>>>(p); break;
-        default: norm_step_kernel<T, V, 8><<<rows, threads, 0, st>>>(p); break;
+        case 8: norm_step_kernel<T, V, 8><<<rows, threads, 0, st>>>(p); break;
+        default:
+            if constexpr (V == 1) norm_step_kernel<T, V, 32><<<rows, threads, 0, st>>>(p);
+            break;
     }
     MYNN_LAUNCH_OK("norm_step_kernel");
     return MYNN_OK;

@@ -411,3 +411,85 @@ def tp_reduce_norm(group: TpGroup, buffer: int, x, weight, eps: float, workspace
 
 def tp_check(group: TpGroup):
     ffi.check(ffi.lib().mynn_b200_tp_check(_stream(), ctypes.byref(group.c)))
+
+
+# ---- operators of the block decoder -----------------------------------------------------------------------------------
+def layer_norm(x, weight, bias, eps, out_dtype=torch.float32):
+    """(x - mean) / sqrt(var + eps) * weight + bias over the last axis of f32 x [rows, W]."""
+    out = torch.empty(x.shape, dtype=out_dtype, device=x.device)
+    ffi.check(ffi.lib().mynn_b200_layer_norm(_stream(), _ptr(out), _ptr(x), _ptr(weight), _ptr(bias), eps, x.shape[0], x.shape[1], _dt(out)))
+    return out
+
+
+def residual_layer_norm(x, sub, post, mult, eps, extra=None, norm=None):
+    """x += mult * LN(sub; post) (+ extra), in place; returns LN(x; norm) in sub's dtype, or None."""
+    out = torch.empty_like(sub) if norm is not None else None
+    w, b = norm if norm is not None else (None, None)
+    ffi.check(ffi.lib().mynn_b200_residual_layer_norm(_stream(), _ptr(x), _ptr(sub), _ptr(post[0]), _ptr(post[1]), mult, _ptr(extra), _ptr(w), _ptr(b),
+                                                      _ptr(out), eps, x.shape[0], x.shape[1], _dt(sub)))
+    return out
+
+
+def short_conv_append(proj, past_dev, k_cache, v_cache, heads, conv=None, history=None, cos=None, sin=None):
+    """proj [B, S, C] -> q [B, heads, S, D], the new rows appended to the rings k_cache / v_cache [B, G, rows, D | E] and
+    ``history`` [B, rows, C]; conv f32 [taps, C], cos / sin f32 [positions, rotated / 2]; past_dev int32 on the device."""
+    B, S, C = proj.shape
+    G, D, E = k_cache.shape[1], k_cache.shape[3], v_cache.shape[3]
+    q = torch.empty(B, heads, S, D, dtype=proj.dtype, device=proj.device)
+    ffi.check(ffi.lib().mynn_b200_short_conv_append(
+        _stream(), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(history), _ptr(proj), _ptr(conv), _ptr(cos), _ptr(sin), B, S, heads, G, D, E,
+        conv.shape[0] if conv is not None else 0, 2 * cos.shape[1] if cos is not None else 0, k_cache.shape[2],
+        history.shape[1] if history is not None else 0, _ptr(past_dev), _dt(proj)))
+    return q
+
+
+def window_attention(q, k_cache, v_cache, scale, active, window=0, softcap=0.0, plain=False):
+    """q [B, Hq, Sq, D] at positions active - Sq .. active - 1 over ring caches [B, G, rows, D | E]; returns [B, Sq, Hq, E]."""
+    B, Hq, Sq, D = q.shape
+    G, rows, E = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
+    out = torch.empty(B, Sq, Hq, E, dtype=q.dtype, device=q.device)
+    ws = attention_workspace(B, Hq, G, D, rows, q.device)
+    ffi.check(ffi.lib().mynn_b200_window_attention(_stream(), _ptr(out), _ptr(q), _ptr(k_cache), _ptr(v_cache), scale, softcap, window, B, Hq, G, Sq, D, E,
+                                                   rows, active, None, _dt(q), _ptr(ws), ws.numel() * ws.element_size(), int(plain)))
+    return out
+
+
+class MoeRouting:
+    """Expert choice of M tokens from f32 logits [M, experts] and the products over the chosen experts."""
+
+    def __init__(self, logits, top, groups=1, groups_keep=1):
+        self.M, self.experts = logits.shape
+        self.top = top
+        n = ffi.lib().mynn_b200_moe_workspace_bytes(self.M, self.experts, top)
+        self.workspace = torch.zeros(n, dtype=torch.uint8, device=logits.device)
+        self.weights = torch.empty(self.M, top, dtype=torch.float32, device=logits.device)
+        self.chosen = torch.empty(self.M, top, dtype=torch.int32, device=logits.device)
+        ffi.check(ffi.lib().mynn_b200_moe_route(_stream(), _ptr(self.workspace), n, _ptr(self.weights), _ptr(self.chosen), _ptr(logits), self.M,
+                                                self.experts, top, groups, groups_keep))
+
+    def rows(self):
+        """[M, top]: the routed row (place in expert order) of every (token, slot) pair."""
+        off = 4096 + -(-self.M * self.top * 4 // 16) * 16
+        return self.workspace[off:off + self.M * self.top * 4].view(torch.int32).view(self.M, self.top)
+
+    def matmul(self, act, w, gather, glu=False, out_dtype=None, tensor_core=True):
+        """act [M | M * top, K] times the experts' blocks w [experts, N | 2 N, K] -> [M * top, N] in expert order."""
+        N, K = w.shape[1] // (2 if glu else 1), w.shape[2]
+        out = torch.empty(self.M * self.top, N, dtype=out_dtype or act.dtype, device=act.device)
+        gw = torch.empty(self.M * self.top, K, dtype=act.dtype, device=act.device) if gather and tensor_core else None
+        status = torch.zeros(1, dtype=torch.int32, device=act.device) if tensor_core else None
+        ffi.check(ffi.lib().mynn_b200_moe_matmul(_stream(), _ptr(out), _ptr(act), _ptr(w), _ptr(self.workspace), _ptr(gw), self.M, N, K, self.experts,
+                                                 self.top, int(gather), int(glu), _dt(act), _dt(out), _ptr(status)))
+        self.status = status
+        return out
+
+
+def dense_matmul(act, w, glu=False, out=None, out_dtype=None, status=None):
+    """act [M, K] times w [N, K] (glu: [2 N, K], gate rows first, out = silu(gate) * up).  status: int32 word of the bounded waits;
+    without it the tensor-core kernel is not used."""
+    N = w.shape[0] // (2 if glu else 1)
+    if out is None:
+        out = torch.empty(act.shape[0], N, dtype=out_dtype or act.dtype, device=act.device)
+    ffi.check(ffi.lib().mynn_b200_dense_matmul(_stream(), _ptr(out), _ptr(act), _ptr(w), act.shape[0], N, act.shape[1], _dt(act), _dt(out), int(glu),
+                                               _ptr(status)))
+    return out
