@@ -93,6 +93,26 @@ __device__ __forceinline__ float fast_rcp(float x) {
     return y;
 }
 
+// Raw scores -> capped scores in log2 units, cap2 tanh(.) = cap2 - 2 cap2 / (1 + 2^(cap_k s)), four at a time: one reciprocal of the
+// product of the four denominators serves all of them, which keeps the special-function unit at 1.25 instead of 2 operations per
+// score.  The exponent is held below 30 (there the quotient is below f32 resolution), so the product stays finite.
+template <int N>
+__device__ __forceinline__ void soft_cap_log2(float (&s)[N], float cap2, float cap_k) {
+    static_assert(N % 4 == 0, "four at a time");
+    const float m2 = -2.f * cap2;
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+        float d[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) d[j] = 1.f + fast_exp2(fminf(s[i + j] * cap_k, 30.f));
+        const float ab = d[0] * d[1], cd = d[2] * d[3], r = m2 * fast_rcp(ab * cd), rab = r * cd, rcd = r * ab;
+        s[i] = fmaf(rab, d[1], cap2);
+        s[i + 1] = fmaf(rab, d[0], cap2);
+        s[i + 2] = fmaf(rcd, d[3], cap2);
+        s[i + 3] = fmaf(rcd, d[2], cap2);
+    }
+}
+
 // One lane polls, the whole warp learns the outcome (tcgen05.ld / st below need the warp to stay converged).
 __device__ __forceinline__ bool warp_wait(uint64_t *bar, uint32_t parity, const int *abort_flag) {
     int ok = 1;
@@ -292,10 +312,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tc_fence_before();
             if (!p.p_tmem) warp_arrive(&s_empty[sb]);  // the rows are in registers: the S buffer may take tile j + 2
 
-            if (capped) {
-#pragma unroll
-                for (int i = 0; i < HC; i++) s[i] = fmaf(-2.f * p.cap2, fast_rcp(1.f + fast_exp2(s[i] * p.cap_k)), p.cap2);
-            }
+            if (capped) soft_cap_log2(s, p.cap2, p.cap_k);
             if (col0 + HC > bound) {  // only the diagonal and the last tile carry masked columns
 #pragma unroll
                 for (int i = 0; i < HC; i++)
@@ -625,10 +642,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
 #pragma unroll
             for (int c = 0; c < kTcCols / 32; c++) tmem_ld32(t_lane + colS + c * 32, reinterpret_cast<uint32_t *>(s) + c * 32);
             tmem_ld_wait();
-            if (capped) {
-#pragma unroll
-                for (int i = 0; i < kTcCols; i++) s[i] = fmaf(-2.f * p.cap2, fast_rcp(1.f + fast_exp2(s[i] * p.cap_k)), p.cap2);
-            }
+            if (capped) soft_cap_log2(s, p.cap2, p.cap_k);
             if (kv0 + kTcCols > bound) {  // only the diagonal and the last tile carry masked columns
 #pragma unroll
                 for (int i = 0; i < kTcCols; i++)

@@ -109,6 +109,7 @@ __global__ void __launch_bounds__(256) dense_tile_kernel(const GemmView g) {
 // grid (ceil(N / (16 RT)), groups), 256 threads.  RT: 16-row weight tiles per warp (with GLU: one gate and one up tile, RT == 1).
 // MT: groups of 8 activation rows taken at a time; a group with more rows than 8 MT passes over its weights again (from L2).
 constexpr int kStreamWarps = 8;
+constexpr unsigned kPrefetchCtas = 3 * 148;
 template <typename T, typename O, int MT, int RT, bool GLU>
 __global__ void __launch_bounds__(kStreamWarps * 32, MT * RT * (GLU ? 2 : 1) <= 4 ? 2 : 1) dense_stream_kernel(const GemmView g) {
     constexpr int WT = GLU ? 2 : RT;  // weight tiles of a warp
@@ -116,11 +117,21 @@ __global__ void __launch_bounds__(kStreamWarps * 32, MT * RT * (GLU ? 2 : 1) <= 
     __shared__ float red[kStreamWarps][WT * 16][MT * 8 + 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, t = lane & 3;
     pdl_trigger();
+    const int n0 = blockIdx.x * 16 * (GLU ? 1 : RT);
+    if (!g.off && gridDim.x <= kPrefetchCtas) {
+        // launched as a programmatic dependent: the weights of this CTA travel to L2 while the kernel in front of it still runs
+        // (a CTA of a later wave starts long after that, for it the prefetch would only be one more request)
+        const size_t line = 128 / sizeof(T), total = (size_t)min(16 * (GLU ? 1 : RT), g.N - n0) * g.K;
+        const T *w0 = reinterpret_cast<const T *>(g.w) + (size_t)n0 * g.K;
+        for (size_t i = threadIdx.x * line; i < total; i += kStreamWarps * 32 * line) {
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(w0 + i));
+            if constexpr (GLU) asm volatile("prefetch.global.L2 [%0];" ::"l"(w0 + (size_t)g.N * g.K + i));
+        }
+    }
     pdl_wait();
     int e, r0, cnt;
     if (!group_rows(g, blockIdx.y, e, r0, cnt)) return;
     const T *act = reinterpret_cast<const T *>(g.act), *w = reinterpret_cast<const T *>(g.w) + (size_t)e * (GLU ? 2 : 1) * g.N * g.K;
-    const int n0 = blockIdx.x * 16 * (GLU ? 1 : RT);
     const T *wp[WT][2];  // this lane's two rows of every tile; rows past N repeat the last one and are not stored
 #pragma unroll
     for (int i = 0; i < WT; i++)
@@ -202,11 +213,20 @@ static int run_stream(cudaStream_t st, const GemmView &v, int rows, int groups, 
     const int mt = rows <= 8 ? 1 : rows <= 16 ? 2 : 4;
     const bool wide = !glu && (mt > 1 || v.N >= 16 * 148 * 4) && v.N >= 32 * 100;
     const dim3 grid((v.N + (wide ? 31 : 15)) / (wide ? 32 : 16), groups);
-#define RUN(MT)                                                                              \
-    {                                                                                        \
-        if (glu) dense_stream_kernel<T, O, MT, 1, true><<<grid, kStreamWarps * 32, 0, st>>>(v); \
-        else if (wide) dense_stream_kernel<T, O, MT, 2, false><<<grid, kStreamWarps * 32, 0, st>>>(v); \
-        else dense_stream_kernel<T, O, MT, 1, false><<<grid, kStreamWarps * 32, 0, st>>>(v);  \
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = dim3(kStreamWarps * 32);
+    cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;  // may start (and fetch weights) while its predecessor drains
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+#define RUN(MT)                                                                                            \
+    {                                                                                                      \
+        if (glu) MYNN_CUDA_OK(cudaLaunchKernelEx(&cfg, dense_stream_kernel<T, O, MT, 1, true>, v));        \
+        else if (wide) MYNN_CUDA_OK(cudaLaunchKernelEx(&cfg, dense_stream_kernel<T, O, MT, 2, false>, v)); \
+        else MYNN_CUDA_OK(cudaLaunchKernelEx(&cfg, dense_stream_kernel<T, O, MT, 1, false>, v));           \
     }
     if (mt == 1) RUN(1) else if (mt == 2) RUN(2) else RUN(4)
 #undef RUN

@@ -1,8 +1,8 @@
 // The step between the q/k/v projection and attention in a layer with short convolutions: causal convolution over time on every
 // projected channel, rotation of q and k, and the append to the ring caches, in one launch.
 //
-// A thread owns 8 neighbouring channels of one token (16-byte accesses; a scalar form covers sizes that are not multiples
-// of 8) and reads the taps of the earlier tokens from the projection of the same step or, for the first taps - 1 tokens, from the
+// A thread owns 8 neighbouring channels of one or four tokens (16-byte accesses; a scalar form covers sizes that are not multiples
+// of 8 and more than four taps) and reads the taps of the earlier tokens from the projection of the same step or, for the first taps - 1 tokens, from the
 // ring that keeps the projections of the last hist_rows positions.  The rotation pairs dimensions 2i and 2i + 1, so a pair never
 // leaves its thread.  New projections enter the ring in the same launch when the step is short enough that no slot read here can
 // be one written here (always for a decode step); longer steps append their tail with a second small kernel.
@@ -25,69 +25,88 @@ __device__ __forceinline__ const T *conv_source(const ConvStep &p, int b, int s,
     return reinterpret_cast<const T *>(p.hist) + ((size_t)b * p.hist_rows + pos % p.hist_rows) * C;
 }
 
-template <typename T>
-__global__ void __launch_bounds__(256) conv_step_vec_kernel(const ConvStep p, int write_hist) {
+// grid (channel groups of 8 / 128, B * ceil(S / TPT)), 128 threads.  A thread takes TPT tokens in a row: its weights stay in registers
+// and every projection row is read once for all the taps it takes part in.
+template <typename T, int TAPS, int TPT>
+__global__ void __launch_bounds__(128) conv_step_vec_kernel(const ConvStep p, int write_hist) {
     pdl_trigger();
     pdl_wait();
-    const int Cq = p.Hq * p.D, Ck = p.G * p.D, Cv = p.G * p.E, C = Cq + Ck + Cv;
-    const int per = C >> 3;
-    const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (idx >= (long long)p.B * p.S * per) return;
-    const int row = (int)(idx / per), c = (int)(idx - (long long)row * per) << 3;
-    const int b = row / p.S, s = row - b * p.S;
-    const int past = *p.past, pos = past + s;
-    float y[8] = {};
-    const uint4 own = *reinterpret_cast<const uint4 *>(reinterpret_cast<const T *>(p.proj) + (size_t)row * C + c);
-    auto add = [&](const uint4 &r, const float *w) {
-        const T *e = reinterpret_cast<const T *>(&r);
-        const float4 w0 = *reinterpret_cast<const float4 *>(w), w1 = *reinterpret_cast<const float4 *>(w + 4);
-        y[0] += w0.x * to_f32<T>(e[0]), y[1] += w0.y * to_f32<T>(e[1]), y[2] += w0.z * to_f32<T>(e[2]), y[3] += w0.w * to_f32<T>(e[3]);
-        y[4] += w1.x * to_f32<T>(e[4]), y[5] += w1.y * to_f32<T>(e[5]), y[6] += w1.z * to_f32<T>(e[6]), y[7] += w1.w * to_f32<T>(e[7]);
-    };
-    if (p.taps) {
-        for (int j = 0; j + 1 < p.taps; j++) {
-            bool zero;
-            const T *src = conv_source<T>(p, b, s, p.taps - 1 - j, past, C, zero);
-            if (!zero) add(*reinterpret_cast<const uint4 *>(src + c), p.w + (size_t)j * C + c);
-        }
-        add(own, p.w + (size_t)(p.taps - 1) * C + c);
-        if (write_hist && s >= p.S - p.hist_rows)
-            *reinterpret_cast<uint4 *>(reinterpret_cast<T *>(p.hist) + ((size_t)b * p.hist_rows + pos % p.hist_rows) * C + c) = own;
-    } else {
-        const T *e = reinterpret_cast<const T *>(&own);
+    const int Cq = p.Hq * p.D, Ck = p.G * p.D, C = Cq + Ck + p.G * p.E;
+    const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
+    if (c >= C) return;
+    const int groups = (p.S + TPT - 1) / TPT, b = blockIdx.y / groups, s0 = (blockIdx.y - b * groups) * TPT;
+    const int past = *p.past;
+    constexpr int LAG = TAPS > 0 ? TAPS - 1 : 0;
+    uint4 raw[TPT + LAG];  // rows s0 - LAG .. s0 + TPT - 1
 #pragma unroll
-        for (int i = 0; i < 8; i++) y[i] = to_f32<T>(e[i]);
+    for (int i = 0; i < TPT + LAG; i++) {
+        raw[i] = make_uint4(0u, 0u, 0u, 0u);
+        const int s = s0 + i - LAG;
+        if (s < p.S) {
+            bool zero;
+            const T *src = conv_source<T>(p, b, s, 0, past, C, zero);
+            if (!zero) raw[i] = *reinterpret_cast<const uint4 *>(src + c);
+        }
     }
+    float w[TAPS > 0 ? TAPS : 1][8];
+#pragma unroll
+    for (int j = 0; j < TAPS; j++) {
+        const float4 a = *reinterpret_cast<const float4 *>(p.w + (size_t)j * C + c), d = *reinterpret_cast<const float4 *>(p.w + (size_t)j * C + c + 4);
+        w[j][0] = a.x, w[j][1] = a.y, w[j][2] = a.z, w[j][3] = a.w, w[j][4] = d.x, w[j][5] = d.y, w[j][6] = d.z, w[j][7] = d.w;
+    }
+    // where token 0 of the sequence's step goes, and how far apart tokens are
+    int d, rows = 0;
     T *dst;
-    int d;
     if (c < Cq) {
         const int h = c / p.D;
         d = c - h * p.D;
-        dst = reinterpret_cast<T *>(p.q_out) + (((size_t)b * p.Hq + h) * p.S + s) * p.D + d;
+        dst = reinterpret_cast<T *>(p.q_out) + ((size_t)b * p.Hq + h) * p.S * p.D + d;
     } else if (c < Cq + Ck) {
         const int h = (c - Cq) / p.D;
         d = c - Cq - h * p.D;
-        dst = reinterpret_cast<T *>(p.k_cache) + (((size_t)b * p.G + h) * p.cache_rows + pos % p.cache_rows) * p.D + d;
+        rows = p.cache_rows;
+        dst = reinterpret_cast<T *>(p.k_cache) + ((size_t)b * p.G + h) * rows * p.D + d;
     } else {
         const int h = (c - Cq - Ck) / p.E;
-        d = c - Cq - Ck - h * p.E;
-        dst = reinterpret_cast<T *>(p.v_cache) + (((size_t)b * p.G + h) * p.cache_rows + pos % p.cache_rows) * p.E + d;
+        rows = p.cache_rows;
+        dst = reinterpret_cast<T *>(p.v_cache) + ((size_t)b * p.G + h) * rows * p.E + (c - Cq - Ck - h * p.E);
         d = 1 << 30;  // values are not rotated
     }
-    if (d < p.rot_dims) {
-        const size_t tab = (size_t)pos * (p.rot_dims >> 1) + (d >> 1);
+    const int width = c < Cq + Ck ? p.D : p.E;
 #pragma unroll
-        for (int i = 0; i < 4; i++) {
-            if (d + 2 * i >= p.rot_dims) break;
-            const float cs = p.cos_t[tab + i], sn = p.sin_t[tab + i], u = y[2 * i], v = y[2 * i + 1];
-            y[2 * i] = rope_low(u, v, cs, sn);
-            y[2 * i + 1] = rope_high(u, v, cs, sn);
+    for (int t = 0; t < TPT; t++) {
+        const int s = s0 + t, pos = past + s;
+        if (s >= p.S) break;
+        float y[8] = {};
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) {
+                const T *e = reinterpret_cast<const T *>(&raw[t + j]);
+#pragma unroll
+                for (int i = 0; i < 8; i++) y[i] += w[j][i] * to_f32<T>(e[i]);
+            }
+            if (write_hist && s >= p.S - p.hist_rows)
+                *reinterpret_cast<uint4 *>(reinterpret_cast<T *>(p.hist) + ((size_t)b * p.hist_rows + pos % p.hist_rows) * C + c) = raw[t + LAG];
+        } else {
+            const T *e = reinterpret_cast<const T *>(&raw[t]);
+#pragma unroll
+            for (int i = 0; i < 8; i++) y[i] = to_f32<T>(e[i]);
         }
-    }
-    T o[8];
+        if (d < p.rot_dims) {
+            const size_t tab = (size_t)pos * (p.rot_dims >> 1) + (d >> 1);
 #pragma unroll
-    for (int i = 0; i < 8; i++) o[i] = from_f32<T>(y[i]);
-    *reinterpret_cast<uint4 *>(dst) = *reinterpret_cast<const uint4 *>(o);
+            for (int i = 0; i < 4; i++) {
+                if (d + 2 * i >= p.rot_dims) break;
+                const float cs = p.cos_t[tab + i], sn = p.sin_t[tab + i], u = y[2 * i], v = y[2 * i + 1];
+                y[2 * i] = rope_low(u, v, cs, sn);
+                y[2 * i + 1] = rope_high(u, v, cs, sn);
+            }
+        }
+        T o[8];
+#pragma unroll
+        for (int i = 0; i < 8; i++) o[i] = from_f32<T>(y[i]);
+        *reinterpret_cast<uint4 *>(dst + (size_t)(rows ? pos % rows : s) * width) = *reinterpret_cast<const uint4 *>(o);
+    }
 }
 
 // any sizes and dtypes: one channel per thread; a rotated channel computes its partner's convolution as well
@@ -150,6 +169,39 @@ __global__ void __launch_bounds__(256) conv_history_kernel(const ConvStep p, int
         reinterpret_cast<const T *>(p.proj)[((size_t)b * p.S + s) * C + c];
 }
 
+template <typename T>
+static int launch_history(cudaStream_t st, const ConvStep &p, int C, int fused) {
+    if (!p.taps || fused) return MYNN_OK;
+    const int keep = p.S < p.hist_rows ? p.S : p.hist_rows;
+    conv_history_kernel<T><<<(unsigned)(((long long)p.B * keep * C + 255) / 256), 256, 0, st>>>(p, keep, C);
+    MYNN_LAUNCH_OK("conv_history_kernel");
+    return MYNN_OK;
+}
+
+template <typename T, int TPT>
+static int run_conv_vec(cudaStream_t st, const ConvStep &p, int C, int fused) {
+    const dim3 grid((C / 8 + 127) / 128, p.B * ((p.S + TPT - 1) / TPT));
+    switch (p.taps) {
+        case 0: conv_step_vec_kernel<T, 0, TPT><<<grid, 128, 0, st>>>(p, fused); break;
+        case 1: conv_step_vec_kernel<T, 1, TPT><<<grid, 128, 0, st>>>(p, fused); break;
+        case 2: conv_step_vec_kernel<T, 2, TPT><<<grid, 128, 0, st>>>(p, fused); break;
+        case 3: conv_step_vec_kernel<T, 3, TPT><<<grid, 128, 0, st>>>(p, fused); break;
+        default: conv_step_vec_kernel<T, 4, TPT><<<grid, 128, 0, st>>>(p, fused); break;
+    }
+    MYNN_LAUNCH_OK("conv_step_vec_kernel");
+    return launch_history<T>(st, p, C, fused);
+}
+
+template <typename T>
+static int launch_conv_vec(cudaStream_t st, const ConvStep &p, int C, int fused) {
+    // the grid's second dimension holds 65535 token groups
+    if (p.S >= 8 || (long long)p.B * p.S > 65535) {
+        if ((long long)p.B * ((p.S + 3) / 4) > 65535) return fail(MYNN_E_UNSUPPORTED, "conv_step: %d x %d tokens in one step", p.B, p.S);
+        return run_conv_vec<T, 4>(st, p, C, fused);
+    }
+    return run_conv_vec<T, 1>(st, p, C, fused);
+}
+
 int launch_conv_step(cudaStream_t st, int dtype, const ConvStep &p) {
     if (p.B <= 0 || p.S <= 0 || p.Hq <= 0 || p.G <= 0 || p.D <= 0 || p.E <= 0 || p.cache_rows <= 0 || p.taps < 0 || p.rot_dims < 0 || p.rot_dims > p.D ||
         p.rot_dims % 2)
@@ -159,24 +211,15 @@ int launch_conv_step(cudaStream_t st, int dtype, const ConvStep &p) {
     if (!p.proj || !p.q_out || !p.k_cache || !p.v_cache || !p.past || (p.rot_dims && (!p.cos_t || !p.sin_t))) return fail(MYNN_E_ARG, "conv_step: null pointer");
     const int C = p.Hq * p.D + p.G * (p.D + p.E);
     const uintptr_t a = (uintptr_t)p.proj | (uintptr_t)p.hist | (uintptr_t)p.w | (uintptr_t)p.q_out | (uintptr_t)p.k_cache | (uintptr_t)p.v_cache;
-    const bool vec = dtype != MYNN_F32 && p.D % 8 == 0 && p.E % 8 == 0 && a % 16 == 0;
+    const bool vec = dtype != MYNN_F32 && p.D % 8 == 0 && p.E % 8 == 0 && a % 16 == 0 && p.taps <= 4;
     const int fused = p.S + p.taps - 1 <= p.hist_rows;  // no ring slot is both read and written by this step
-    const long long n = (long long)p.B * p.S * (vec ? C / 8 : C);
-    const unsigned blocks = (unsigned)((n + 255) / 256);
-    if (vec) {
-        if (dtype == MYNN_BF16) conv_step_vec_kernel<__nv_bfloat16><<<blocks, 256, 0, st>>>(p, fused);
-        else conv_step_vec_kernel<__half><<<blocks, 256, 0, st>>>(p, fused);
-        MYNN_LAUNCH_OK("conv_step_vec_kernel");
-    } else {
+    if (vec) return dtype == MYNN_BF16 ? launch_conv_vec<__nv_bfloat16>(st, p, C, fused) : launch_conv_vec<__half>(st, p, C, fused);
+    const unsigned blocks = (unsigned)(((long long)p.B * p.S * C + 255) / 256);
+    {
         MYNN_DISPATCH_DTYPE(dtype, T, { conv_step_kernel<T><<<blocks, 256, 0, st>>>(p, fused); });
         MYNN_LAUNCH_OK("conv_step_kernel");
     }
-    if (p.taps && !fused) {
-        const int keep = p.S < p.hist_rows ? p.S : p.hist_rows;
-        const unsigned hb = (unsigned)(((long long)p.B * keep * C + 255) / 256);
-        MYNN_DISPATCH_DTYPE(dtype, T, { conv_history_kernel<T><<<hb, 256, 0, st>>>(p, keep, C); });
-        MYNN_LAUNCH_OK("conv_history_kernel");
-    }
+    MYNN_DISPATCH_DTYPE(dtype, T, { return launch_history<T>(st, p, C, fused); });
     return MYNN_OK;
 }
 

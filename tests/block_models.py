@@ -29,7 +29,7 @@ def config(width, vocab, layers, loop=None, embed=2.0, mult=0.7, eps=1e-5):
 def mixed():
     """Layers of different sizes, none of which the tuned attention kernels take; one without a feed-forward, a loop of two."""
     return config(72, 101, [
-        layer(6, 2, 24, 40, 19, 3, rot(8, 500.0, (8.0, 1.0, 4.0, 64.0)), moe=(24, 6, 2, 3, 2)),
+        layer(6, 2, 24, 40, 19, 3, rot(8, 500.0, (8.0, 1.0, 4.0, 64.0)), moe=(24, 6, 2, 3, 1)),
         layer(4, 4, 12, 12, 33, 2, rot(12), softcap=4.0, moe=(16, 4, 3, 1, 1)),
         layer(3, 1, 32, 16, 7, 5, rot(6, 100.0)),
         layer(2, 2, 16, 24, 50, 1, rot(16, 1e6), moe=(40, 9, 1, 3, 1)),
@@ -40,13 +40,22 @@ def even_group():
     """Head size 64, two query heads per kv head."""
     return config(128, 160, [layer(4, 2, 64, 64, 50, 4, rot(32, 1e4, (4.0, 1.0, 4.0, 128.0)), moe=(48, 8, 2, 4, 2)),
                              layer(8, 2, 64, 64, 131, 3, rot(64), moe=(32, 8, 3, 2, 1))],
-                  loop={"start": 0, "stop": 1, "times": 3}, embed=4.0, mult=0.4, eps=1e-6)
+                  loop={"start": 0, "stop": 1, "times": 3}, embed=1.0, mult=0.8, eps=1e-6)
 
 
 def odd_group():
     """Head size 128, three query heads per kv head, no loop."""
     return config(96, 90, [layer(3, 1, 128, 128, 140, 2, rot(16), softcap=30.0, moe=(64, 5, 2, 1, 1)),
-                           layer(6, 2, 128, 128, 16, 4, rot(128, 1e5), moe=(16, 12, 4, 6, 3))], mult=1.0, embed=1.0)
+                           layer(6, 2, 128, 128, 16, 4, rot(128, 1e5), moe=(16, 12, 4, 6, 3))], mult=0.7, embed=1.0)
+
+
+def all_chosen(cfg, experts=3):
+    """The same model with few experts that every token uses: no choice that 16-bit rounding could tip, so that 16-bit logits can be
+    held to a tight limit."""
+    for e in cfg["layers"]:
+        if e["mlp"]:
+            e["mlp"]["router"].update(experts=experts, top=experts, groups={"count": 1, "keep": 1})
+    return cfg
 
 
 ALL = {"mixed": mixed, "even_group": even_group, "odd_group": odd_group}

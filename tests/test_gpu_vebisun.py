@@ -16,23 +16,24 @@ from my_nn_engine_b200.session import GenerateOptions, LlmSession  # noqa: E402
 from oracle import ref_vebisun as R  # noqa: E402
 from tests import block_models as bm  # noqa: E402
 
-LIMIT = {"f32": 2e-5, "bf16": 6e-2}
+LIMIT = {"f32": 2e-5, "bf16": 4e-2}
 LENGTH = 330
 _cache = {}
 
 
-def case(name):
-    """(cfg, state, tokens, oracle logits [LENGTH, vocab]) of a small model, computed once."""
-    if name not in _cache:
-        cfg = bm.ALL[name]()
+def case(name, dtype="f32"):
+    """(cfg, state, tokens, oracle logits [LENGTH, vocab]) of a small model, computed once; for bf16 the variant without an expert
+    choice to tip."""
+    if (name, dtype) not in _cache:
+        cfg = bm.ALL[name]() if dtype == "f32" else bm.all_chosen(bm.ALL[name]())
         state = bm.weights(cfg, seed=len(name))
         toks = np.random.default_rng(5).integers(0, cfg["vocab"], LENGTH).tolist()
-        _cache[name] = cfg, state, toks, R.forward(cfg, bm.as_numpy(state), toks)
-    return _cache[name]
+        _cache[name, dtype] = cfg, state, toks, R.forward(cfg, bm.as_numpy(state), toks)
+    return _cache[name, dtype]
 
 
-def model_of(name, dtype, **kw):
-    cfg, state, _, _ = case(name)
+def model_of(name, dtype, routed=False, **kw):
+    cfg, state, _, _ = case(name, "f32" if routed else dtype)
     kw.setdefault("max_seq_len", LENGTH + 20)
     return vebisun.build(cfg, state, dtype=dtype, **kw)
 
@@ -58,24 +59,34 @@ def portions(total, sizes):
 def check(got, want, dtype, what=""):
     e = bm.rel_error(got, want)
     worst = int(e.argmax())
-    # bf16: a router that is nearly undecided may fall either way; a wrong mechanism shows in far more rows
-    share = (e > LIMIT[dtype]).mean()
-    assert share <= (0.0 if dtype == "f32" else 0.03), f"{what}: {share:.3f} of the rows over the limit, worst {e[worst]:.3g} at {worst}, first at {int(np.argmax(e > LIMIT[dtype]))}"
+    assert e[worst] <= LIMIT[dtype], f"{what}: {(e > LIMIT[dtype]).mean():.3f} of the rows over the limit, worst {e[worst]:.3g} at {worst}, first at {int(np.argmax(e > LIMIT[dtype]))}"
 
 
 @pytest.mark.parametrize("dtype", ["f32", "bf16"])
 @pytest.mark.parametrize("name", sorted(bm.ALL))
 @pytest.mark.parametrize("sizes", [[LENGTH], [1], [2], [3, 64, 2, 17, 1, 5], [100, 129], [16]], ids=str)
 def test_portions(name, dtype, sizes):
-    _, _, toks, want = case(name)
+    _, _, toks, want = case(name, dtype)
     m = model_of(name, dtype, max_prefill=LENGTH if sizes == [LENGTH] else 130)
     check(run(m, toks, portions(LENGTH, sizes)), want, dtype, f"{name} {sizes}")
     m.close()
 
 
+@pytest.mark.parametrize("name", sorted(bm.ALL))
+@pytest.mark.parametrize("sizes", [[LENGTH], [1], [40, 3]], ids=str)
+def test_routed_experts_in_16_bits(name, sizes):
+    """With a real expert choice 16-bit rounding tips a close call now and then, and the rows that look at such a token follow it: the
+    bulk of the rows has to agree."""
+    _, _, toks, want = case(name)
+    m = model_of(name, "bf16", routed=True, max_prefill=LENGTH)
+    e = bm.rel_error(run(m, toks, portions(LENGTH, sizes)), want)
+    assert np.median(e) < 2.5e-2 and (e < 0.1).mean() > 0.8, (np.median(e), (e < 0.1).mean())
+    m.close()
+
+
 @pytest.mark.parametrize("dtype", ["f32", "bf16"])
 def test_prompt_then_long_decoding_past_several_ring_turns(dtype):
-    _, _, toks, want = case("mixed")
+    _, _, toks, want = case("mixed", dtype)
     m = model_of("mixed", dtype, max_prefill=8, max_rewind=0)  # rings as short as they can be
     assert min(s[0].shape[2] for s in m.run_states) == 128
     check(run(m, toks, [8, 5] + [1] * (LENGTH - 13)), want, dtype)
@@ -84,7 +95,7 @@ def test_prompt_then_long_decoding_past_several_ring_turns(dtype):
 
 @pytest.mark.parametrize("name", ["even_group", "odd_group"])
 def test_without_a_graph_and_with_the_plain_prefill_kernels(name):
-    _, _, toks, want = case(name)
+    _, _, toks, want = case(name, "bf16")
     m = model_of(name, "bf16", max_prefill=64, use_graph=False)
     ffi.set_option(ffi.OPT_PREFILL_ATTENTION, 0)
     ffi.set_option(ffi.OPT_DECODE_RING, 0)
@@ -100,7 +111,7 @@ def test_without_a_graph_and_with_the_plain_prefill_kernels(name):
 @pytest.mark.parametrize("name", sorted(bm.ALL))
 def test_state_is_given_back_and_used_again(name, dtype):
     """A long sequence, then shorter ones in the same rings: nothing of the earlier one may show, also in its first tokens."""
-    cfg, state, toks, want = case(name)
+    cfg, state, toks, want = case(name, dtype)
     m = model_of(name, dtype, max_prefill=50)
     run(m, toks[::-1], portions(LENGTH, [50]))
     check(run(m, toks[:1], [1]), want[:1], dtype, "one token")
@@ -122,7 +133,7 @@ def test_rewind_within_the_allowed_positions_and_errors():
         m.feed([1], 300)
     with pytest.raises(ffi.MynnError, match="rewind"):
         m.feed([1, 2], 5)
-    check(run(m, toks[:40], [7, 33][:1] + [32, 1]), want[:40], "f32", "a new sequence after an error")
+    check(run(m, toks[:40], [7, 32, 1]), want[:40], "f32", "a new sequence after an error")
     m.close()
 
 
@@ -130,7 +141,7 @@ def test_rewind_within_the_allowed_positions_and_errors():
 @pytest.mark.parametrize("name", ["mixed", "even_group"])
 def test_batch_against_each_alone(name, dtype):
     """Three different sequences side by side (one past length for all, as every model here batches)."""
-    cfg, state, toks, _ = case(name)
+    cfg, state, toks, _ = case(name, dtype)
     rng = np.random.default_rng(9)
     seqs = [toks[:150], rng.integers(0, cfg["vocab"], 150).tolist(), toks[100:250]]
     W = bm.as_numpy(state)
@@ -161,8 +172,8 @@ def test_first_tokens_and_single_token_prompts():
         m.close()
 
 
-def save(tmp_path, name):
-    cfg, state, toks, want = case(name)
+def save(tmp_path, name, dtype="f32"):
+    cfg, state, toks, want = case(name, dtype)
     (tmp_path / "config.json").write_text(json.dumps(cfg))
     write_safetensors(str(tmp_path / "model.safetensors"), state)
     return str(tmp_path), cfg, state, toks, want
@@ -199,7 +210,8 @@ def test_generate_command(tmp_path):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_trace_runner(tmp_path, dtype):
-    d, cfg, state, toks, want = save(tmp_path, "mixed")
+    dt = {"float32": "f32", "bfloat16": "bf16"}[dtype]
+    d, cfg, state, toks, want = save(tmp_path, "mixed", dt)
     out = tmp_path / "out"
     out.mkdir()
     steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:100], "want": [99, 0, 41]}], "end": []},
@@ -211,7 +223,6 @@ def test_trace_runner(tmp_path, dtype):
                        input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=600)
     assert r.returncode == 0, r.stderr
     assert [x for x in r.stdout.splitlines() if x.startswith("done")] == ["done 0", "done 1", "done 2", "done 3"]
-    dt = {"float32": "f32", "bfloat16": "bf16"}[dtype]
 
     def read(n):
         return np.fromfile(out / f"{n}.f32", "<f4").reshape(-1, cfg["vocab"])

@@ -84,7 +84,7 @@ def test_configuration_is_read_in_full():
     spec = vebisun.spec_from_config(bm.mixed())
     a = spec.layers[0]
     assert (a.heads, a.kv_heads, a.dim, a.vdim, a.window, a.conv_taps, a.softcap) == (6, 2, 24, 40, 19, 3, 15.0)
-    assert (a.experts, a.expert_ff, a.top, a.groups, a.groups_keep) == (6, 24, 2, 3, 2)
+    assert (a.experts, a.expert_ff, a.top, a.groups, a.groups_keep) == (6, 24, 2, 3, 1)
     assert a.rotary.scaling.factor == 8.0 and a.channels == 6 * 24 + 2 * 64
     assert spec.layers[2].experts == 0 and spec.loop == (1, 3, 2) and spec.runs() == [0, 1, 2, 1, 2, 3]
     assert (spec.embed_scale, spec.residual_mult, spec.norm_eps) == (2.0, 0.7, 1e-5)
