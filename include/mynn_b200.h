@@ -394,41 +394,72 @@ int mynn_b200_tp_reduce_norm(void *stream, const mynn_b200_tp_group *group, int 
 int mynn_b200_tp_check(void *stream, const mynn_b200_tp_group *group);
 
 /* ---------------------------------------------------------------------------------------------
- * Block decoders: models given as a list of layers, each with its own sizes, over unquantised weights.  No counterpart in the
- * engine.  A layer is
- *     x += residual_mult * LN(mixer(LN(x)));   x += residual_mult * LN(ff(LN(x)))      (ff absent when experts == 0)
- * with x in f32, LN a layer norm with weight and bias, the mixer causal attention (below) and ff a mixture of SiLU-gated
- * experts.  Layers [loop_start, loop_stop) run loop_times times in a row with the same weights and a state per pass; before
- * every pass but the first the embedding output is added to x.  Embedding rows are multiplied by embed_scale; the head is
- * LN, then a product.  Attention: q/k/v projections through a causal convolution over conv_taps tokens per channel, interleaved
- * rotation of the first rot_dims dimensions of q and k, scores attn_scale * q.k through softcap * tanh(. / softcap), the last
- * `window` positions visible.  Experts: softmax router over all experts, groups_keep of `groups` groups by best member, `top`
- * experts, weights not renormalised.
+ * Block decoders: models given as a list of layers, each with its own mixer, feed-forward and sizes, over unquantised weights.  No
+ * counterpart in the engine.  A layer is
+ *     x += residual_mult * N(mixer(N(x)));   x += residual_mult * N(ff(N(x)))      (ff absent when experts == dense_ff == 0)
+ * with x in f32 and N a layer norm with weight and bias (rms_norm == 0) or v / sqrt(mean(v^2) + norm_eps) * weight (rms_norm != 0);
+ * without post_norm the outer N is absent.  Layers [loop_start, loop_stop) run loop_times times in a row with the same weights and
+ * a state per pass; before every pass but the first the embedding output is added to x.  Embedding rows are multiplied by
+ * embed_scale; the head is N, then a product.
+ *
+ * Mixers:
+ *   MYNN_MIX_ATTENTION  causal attention: q/k/v projections through a causal convolution over conv_taps tokens per channel, rotation
+ *       of the first rot_dims dimensions of q and k (rot_halves: dimension i with i + rot_dims / 2, else 2i with 2i + 1), with qk_norm
+ *       each q and k head over its root mean square afterwards, scores attn_scale * q.k through softcap * tanh(. / softcap), the last
+ *       `window` positions visible, and of those the ones in the query's own chunk of `chunk` positions (counted from position 0).
+ *       rot_halves and qk_norm go with conv_taps == 0.
+ *   MYNN_MIX_LATENT     attention through latents: queries N(W_dq h) of q_rank numbers, then W_uq; keys and values W_uk c, W_uv c of
+ *       c = N(W_dkv h), kv_rank numbers per position that all heads share and that alone are cached (both N by root mean square);
+ *       heads of dim / vdim, scores attn_scale * q.k, no positions, the whole past visible.
+ *   MYNN_MIX_MLSTM      matrix memory with exponential gates (mynn_b200_mlstm below), gate_cap, heads of dim / vdim.
+ * Feed-forwards: a mixture of `experts` SiLU-gated experts (softmax router over all experts, groups_keep of `groups` groups by best
+ * member, `top` experts, weights not renormalised), or with dense_ff > 0: W_down f(W_up x), f by ff_act.
  *
  * They are stepped through the entry points above: configure, model_init, model / model_step_device / model_prefill /
- * model_prefill_rows, model_destroy.  Logits are f32.  dtype is that of weights, activations and caches; norms, scores, router,
- * convolution sums and the residual stream are f32 in every dtype.
+ * model_prefill_rows, model_destroy.  Logits are f32.  dtype is that of weights, activations and caches; norms, scores, router, gates,
+ * convolution sums, recurrent state and the residual stream are f32 in every dtype.
  *
- * initializer order: embed [V, H]; per layer norm1 w, b; norm1b w, b; qkv [heads*dim + kv_heads*(dim+vdim), H]; conv f32
- *   [taps, rows of qkv] (NULL without); o [H, heads*vdim]; cos, sin f32 [max_seq_len, rot_dims/2] (NULL without); norm2 w, b;
- *   norm2b w, b; router [experts, H]; gate_up [experts, 2*expert_ff, H] (gate rows, then up rows); down [experts, H, expert_ff]
- *   (these seven NULL without experts); then final norm w, b; head [V, H].  Norm weights f32.
- * session_state order: per layer RUN (a repeated layer counts per pass) K ring [batch, kv_heads, cache_rows, dim], V ring
- *   [batch, kv_heads, cache_rows, vdim], convolution ring [batch, history_rows, rows of qkv] (NULL without), zeroed.  Position p of
- *   a sequence lives in row p % cache_rows resp. p % history_rows.  cache_rows: a multiple of 128, and at least max_seq_len or
- *   window - 1 + max_prefill + max_rewind; history_rows >= conv_taps + max_rewind.
- * past_len of a step is 0 (a new sequence), the number of positions stored, or up to max_rewind fewer than were ever stored. */
+ * initializer order: embed [V, H]; per layer 22 pointers, NULL where a layer has no such thing:
+ *    0-3   norm1 w, b; norm1b (post norm) w, b
+ *    4     projection of the mixer's input: attention [heads*dim + kv_heads*(dim+vdim), H] (q, k, v rows); latent [q_rank + kv_rank, H]
+ *          (dq, dkv rows); mlstm [heads*(2 dim + 2 vdim + 2), H] (q, k, v, output gate, input gate, forget gate rows)
+ *    5     conv f32 [taps, rows of 4]
+ *    6     o [H, heads*vdim]
+ *    7-8   cos, sin f32 [max_seq_len, rot_dims/2]
+ *    9-12  norm2 w, b; norm2b w, b
+ *    13-15 router [experts, H]; gate_up [experts, 2*expert_ff, H] (gate rows, then up rows), dense: up [dense_ff, H];
+ *          down [experts, H, expert_ff], dense: [H, dense_ff]
+ *    16-17 f32 vectors: latent: the weights of the two latents' norms [q_rank], [kv_rank]; mlstm: head norm weight [heads*vdim], gate
+ *          biases [2 heads] (input, forget)
+ *    18-21 latent: W_uq [heads*dim, q_rank], W_uk [heads*dim, kv_rank], W_uk per head transposed [heads, kv_rank, dim],
+ *          W_uv [heads*vdim, kv_rank]
+ * then final norm w, b; head [V, H].  Norm weights f32; biases are NULL with rms_norm.
+ * session_state order: three per layer RUN (a repeated layer counts per pass), zeroed: attention K ring [batch, kv_heads, cache_rows,
+ *   dim], V ring [batch, kv_heads, cache_rows, vdim], convolution ring [batch, history_rows, rows of 4] (NULL without); latent: c
+ *   [batch, cache_rows, kv_rank], NULL, NULL; mlstm f32 memory [batch, heads, dim, vdim], sum [batch, heads, dim], maximum [batch, heads].
+ *   Position p of a sequence lives in row p % cache_rows resp. p % history_rows.  cache_rows: a multiple of 128, and at least
+ *   max_seq_len or (window or chunk) - 1 + max_prefill + max_rewind (0 for mlstm); history_rows >= conv_taps + max_rewind.
+ * past_len of a step is 0 (a new sequence), the number of positions stored, or up to max_rewind fewer than were ever stored.  A model
+ * with a recurrent layer cannot go back: past_len is 0 or the number of positions stored. */
+enum { MYNN_MIX_ATTENTION = 0, MYNN_MIX_LATENT = 1, MYNN_MIX_MLSTM = 2 };
+enum { MYNN_ACT_NONE = 0, MYNN_ACT_SQUARE_RELU = 1 };
 typedef struct mynn_b200_block {
     int32_t heads, kv_heads, dim, vdim;
     int32_t conv_taps, rot_dims;
     int32_t window;  /* 0: the whole past */
     int32_t cache_rows, history_rows;
     int32_t experts, expert_ff, top, groups, groups_keep;
+    int32_t mixer, rot_halves, qk_norm;
+    int32_t chunk;   /* 0: none */
+    int32_t q_rank, kv_rank;
+    int32_t dense_ff, ff_act;
     float attn_scale, softcap; /* softcap 0: none */
+    float gate_cap;
 } mynn_b200_block;
 typedef struct mynn_b200_block_model_config {
     int32_t n_layers, hidden, vocab, max_seq_len, batch, dtype, output_mode, use_graph, max_prefill, max_rewind;
     int32_t loop_start, loop_stop, loop_times; /* loop_times <= 1: no loop */
+    int32_t rms_norm, post_norm;
     float embed_scale, residual_mult, norm_eps;
     const mynn_b200_block *layers;
 } mynn_b200_block_model_config;
@@ -443,6 +474,8 @@ int mynn_b200_layer_norm(void *stream, void *out, const float *x, const float *w
 int mynn_b200_residual_layer_norm(void *stream, float *x, const void *sub, const float *post_weight, const float *post_bias, float mult,
                                   const float *extra, const float *weight, const float *bias, void *out, float eps, int rows, int W,
                                   int dtype);
+/* x += sub (dtype, may be NULL); out = x / sqrt(mean(x^2) + eps) * weight in dtype (may be NULL). */
+int mynn_b200_residual_rms_norm(void *stream, float *x, const void *sub, const float *weight, void *out, float eps, int rows, int W, int dtype);
 /* S new positions *past_dev .. of B sequences: proj [B*S, Hq*D + Hkv*(D+E)] -> causal convolution (f32 [taps, columns of proj]) ->
  * interleaved rotation -> q_out [B, Hq, S, D] and the rings (see above).  S <= cache_rows. */
 int mynn_b200_short_conv_append(void *stream, void *q_out, void *k_cache, void *v_cache, void *history, const void *proj,
@@ -453,6 +486,35 @@ int mynn_b200_short_conv_append(void *stream, void *q_out, void *k_cache, void *
 int mynn_b200_window_attention(void *stream, void *out, const void *q, const void *k, const void *v, float scale, float softcap,
                                int window, int B, int Hq, int Hkv, int Sq, int D, int E, int cache_rows, int active,
                                const int32_t *active_dev, int dtype, void *workspace, size_t workspace_bytes, int plain);
+/* The same with chunks (chunk > 0: nothing before the query's own chunk of that many positions is seen, chunks count from position 0) and, with
+ * head_major, q [Hq, B, Sq, D] and caches [Hkv, B, rows, .]. */
+int mynn_b200_chunk_attention(void *stream, void *out, const void *q, const void *k, const void *v, float scale, float softcap,
+                              int window, int chunk, int head_major, int B, int Hq, int Hkv, int Sq, int D, int E, int cache_rows, int active,
+                              const int32_t *active_dev, int dtype, void *workspace, size_t workspace_bytes, int plain);
+/* The step of mynn_b200_short_conv_append without a convolution: rotation (halves: dimension i with i + rot_dims / 2, else 2i with 2i + 1),
+ * with qk_norm every q and k head v / sqrt(mean(v^2) + eps) afterwards, append. */
+int mynn_b200_rotary_append(void *stream, void *q_out, void *k_cache, void *v_cache, const void *proj, const float *cos_table,
+                            const float *sin_table, int B, int S, int Hq, int Hkv, int D, int E, int rot_dims, int halves, int qk_norm,
+                            float eps, int cache_rows, const int32_t *past_dev, int dtype);
+/* proj [B*S, Q + R] of S new tokens at positions *past_dev ..: both parts over their root mean square, weighted (f32); the first to q_out
+ * [B*S, Q], the second to cache [B, cache_rows, R]. */
+int mynn_b200_latent_append(void *stream, void *q_out, void *cache, const void *proj, const float *q_weight, const float *c_weight, float eps,
+                            int B, int S, int Q, int R, int cache_rows, const int32_t *past_dev, int dtype);
+/* q [B, Sq, H, R] at positions active - Sq .. active - 1 over latents cache [B, cache_rows, R], keys and values at once, causal; out
+ * [B, Sq, H, R].  workspace may be NULL.  plain != 0: the kernel for any sizes. */
+size_t mynn_b200_latent_attention_workspace_bytes(int B, int Sq, int H, int R, int cache_rows);
+int mynn_b200_latent_attention(void *stream, void *out, const void *q, const void *cache, float scale, int B, int Sq, int H, int R, int cache_rows,
+                               int active, const int32_t *active_dev, int dtype, void *workspace, size_t workspace_bytes, int plain);
+/* Matrix memory with exponential gates over S new tokens of B sequences.  proj [B*S, H*(2D + 2E)] (q, k, v, output gate z), gates f32
+ * [B*S, 2H] and gate_bias f32 [2H] (input, forget).  Per head, with q~ = q / sqrt(D), cap(x) = gate_cap tanh(x / gate_cap):
+ *   i = cap(gates_i + bias_i), f = log sigmoid(cap(gates_f + bias_f)), m' = max(f + m, i), a = e^(f + m - m'), w = e^(i - m'),
+ *   S' = a S + w k v^T, n' = a n + w k, o = S'^T q~ / (max(|n'.q~|, e^-m') + 1e-6),
+ *   out = o / sqrt(mean(o^2) + eps) * norm_weight * sigmoid(z)          (out [B*S, H*E], norm_weight f32 [H*E])
+ * State f32 in place: mem [B, H, D, E], sum [B, H, D] (n), top [B, H] (m); taken as zero when *past_dev == 0.  scratch f32 [B*S, H*E];
+ * tickets [B*H], zero before the first use.  form 0: by size, 1: token by token, 2: chunkwise on the tensor cores (16-bit). */
+int mynn_b200_mlstm(void *stream, void *out, float *mem, float *sum, float *top, const void *proj, const float *gates, const float *gate_bias,
+                    const float *norm_weight, float cap, float eps, int B, int S, int H, int D, int E, const int32_t *past_dev, float *scratch,
+                    uint32_t *tickets, int dtype, int form);
 /* Expert choice from f32 logits [M, experts]; the workspace (zeroed before its first use) then describes the (token, slot) rows in expert order
  * for mynn_b200_moe_matmul.  weights_out f32 / experts_out int32 [M, top] may be NULL. */
 size_t mynn_b200_moe_workspace_bytes(int M, int experts, int top);
@@ -462,6 +524,12 @@ int mynn_b200_moe_route(void *stream, void *workspace, size_t workspace_bytes, f
  * status: device word of the bounded waits (NULL keeps the tensor-core kernel off). */
 int mynn_b200_dense_matmul(void *stream, void *out, const void *act, const void *w, int M, int N, int K, int dtype, int out_dtype, int glu,
                            int32_t *status);
+/* The same with more of a product's options: act_fn on the f32 sums; out_f32 (may be NULL): columns from n_main on go there in f32, [M, N - n_main];
+ * out_block > 0: column n of row m at (n / out_block) * out_block_stride + m * ldo + n % out_block of out; batch independent products,
+ * product z of act + z * act_stride (rows lda apart), w + z * N * K, out + z * out_stride.  lda, ldo 0: dense rows. */
+int mynn_b200_dense_matmul_ex(void *stream, void *out, const void *act, const void *w, int M, int N, int K, int dtype, int out_dtype, int act_fn,
+                              float *out_f32, int n_main, int out_block, long long out_block_stride, int lda, int ldo, int batch,
+                              long long act_stride, long long out_stride, int32_t *status);
 /* The same per expert over the M * top routed rows: w [experts, N or 2N, K]; gather: act has one row per token, else one per routed
  * row.  gather_workspace: M * top * K elements (NULL keeps the tensor-core kernel off when gather is set). */
 int mynn_b200_moe_matmul(void *stream, void *out, const void *act, const void *w, void *route_workspace, void *gather_workspace, int M, int N,

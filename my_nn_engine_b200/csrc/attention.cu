@@ -61,7 +61,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     int active = p.active_dev ? *p.active_dev : p.active_host;
     active = max(0, WIN && p.ring_cache ? active : min(active, p.cache_seq));
     // rows [lo, active) are seen; the walk starts at the 16-row tile that holds lo (0 without a window)
-    const int lo = WIN ? max(p.window > 0 ? max(0, active - p.window) : 0, p.ring_cache ? active - p.cache_seq : 0) : 0, walk0 = lo & ~15;
+    const int lo = WIN ? max(active > 0 ? first_visible(active - 1, p.window, p.chunk) : 0, p.ring_cache ? active - p.cache_seq : 0) : 0, walk0 = lo & ~15;
     // whole rounds of the CTA's four warps (64 rows): a split that ends inside a round leaves some warps a tile short
     const int rows_per_split = (((active - walk0 + p.splits - 1) / p.splits) + 16 * kAttnWarps - 1) / (16 * kAttnWarps) * (16 * kAttnWarps);
     const int row_beg = walk0 + split * rows_per_split;
@@ -635,7 +635,7 @@ int mynn::launch_attention(cudaStream_t st, void *out, const void *q, const void
 
 // One query row per sequence over a ring cache with a sliding window and a score soft cap (attention_window.cu picks the kernel).
 bool mynn::window_attention_decode_supported(int dtype, const WindowAttention &w) {
-    return w.D == w.E && w.cache_rows % 16 == 0 && w.workspace &&
+    return w.layout == kByBatch && w.D == w.E && w.cache_rows % 16 == 0 && w.workspace &&
            w.workspace_bytes >= mynn_b200_attention_workspace_bytes(w.B, w.Hq, w.Hkv, w.D, w.cache_rows) &&
            attention_decode_fast_path(w.Sq, w.D, w.Hq, w.Hkv, dtype, w.q, w.k, w.v);
 }
@@ -652,6 +652,7 @@ int mynn::launch_window_attention_decode(cudaStream_t st, int dtype, const Windo
     p.active_dev = w.active;
     int rows_bound = w.active ? w.cache_rows : std::min(w.active_host, w.cache_rows);
     if (w.window > 0) rows_bound = std::min(rows_bound, w.window + 15);
+    if (w.chunk > 0) rows_bound = std::min(rows_bound, w.chunk + 15);
     const bool ring = decode_ring_possible(w.B, w.Hkv, w.cache_rows);
     p.splits = decode_splits(w.B, w.Hkv, rows_bound, 16, decode_ctas_per_sm(ring, w.D));
     p.k_scale = p.v_scale = nullptr;
@@ -659,6 +660,7 @@ int mynn::launch_window_attention_decode(cudaStream_t st, int dtype, const Windo
     p.ascale = nullptr;
     p.status = w.status_word;
     p.window = w.window;
+    p.chunk = w.chunk;
     p.ring_cache = 1;
     p.softcap = w.softcap;
     if (int rc = decode_bind_workspace(p, w.B, w.D, w.workspace, w.workspace_bytes)) return rc;

@@ -38,6 +38,23 @@ __device__ __forceinline__ void mma_kv(float (&c)[4], uint32_t a0, uint32_t a1, 
     }
 }
 
+// Four 8 x 8 matrices of 16-bit elements from shared memory, one row address per lane; `t`: transposed.
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void *p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+                 : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void *p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+                 : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+// 16 bytes global -> shared (cp.async); zeros when !in, without a read
+__device__ __forceinline__ void copy16(void *smem, const void *gmem, bool in) {
+    const int n = in ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem), "r"(n) : "memory");
+}
+
 // pack hi parts of (x, y) into one 32-bit register and the rounding remainders into another
 template <typename T>
 __device__ __forceinline__ void split_pack(float x, float y, uint32_t &hi, uint32_t &lo) {
@@ -79,6 +96,7 @@ struct DecodeParams {
     // Optional (16-bit decode kernel): only the last `window` positions are seen; position p lives in cache row p % cache_seq
     // (ring_cache: `active` may then exceed cache_seq, which is a multiple of 16); scores pass through a soft cap.
     int window = 0, ring_cache = 0;
+    int chunk = 0;  // and none before the query's own chunk of that many positions (counted from position 0)
     float softcap = 0.f;
     int *status = nullptr;  // ring kernel: where a timed-out wait is recorded (null: the library's own word, see attention_check)
 };

@@ -62,7 +62,7 @@ struct TcAttnParams {
     int is_causal, out_bshd;
     uint32_t v_lbo, v_sbo;  // byte offsets of the MN-major V descriptor
     int n_qt, heads_per_grid, B;  // 1-D grid: query tiles x (heads or head pairs) x batch, query tile slowest
-    int window, ring_cache;  // WIN kernels: see WindowAttention (block_ops.cuh); cache_seq is a multiple of 128 then
+    int window, ring_cache, chunk, head_major;  // WIN kernels: see WindowAttention (block_ops.cuh); cache_seq is a multiple of 128 then
     float cap2, cap_k;       // soft cap in log2 units: score -> cap2 - 2 cap2 / (1 + 2^(cap_k * raw)); cap2 == 0: none
     int p_tmem;  // probabilities handed to the second product through tensor memory (over the S columns) instead of shared memory
 };
@@ -167,10 +167,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int last_row = min(q0 + kTcRows, p.Sq) - 1;
     const int kv_end = p.is_causal ? max(0, min(active, past + last_row + 1)) : active;
     // WIN: the walk starts at the tile of the first position that the CTA's first row sees
-    const int kv_beg = WIN ? max(p.window > 0 ? past + q0 + 1 - p.window : 0, max(0, p.ring_cache ? active - p.cache_seq : 0)) / kTcCols * kTcCols : 0;
+    const int kv_beg = WIN ? max(first_visible(max(past + q0, 0), p.window, p.chunk), max(0, p.ring_cache ? active - p.cache_seq : 0)) / kTcCols * kTcCols : 0;
     const int n_tiles = max(0, kv_end - kv_beg + kTcCols - 1) / kTcCols;
-    const int q_row0 = (b * p.Hq + h) * p.Sq + q0;      // row of the Q map
-    const int kv_row0 = (b * p.Hkv + kvh) * p.cache_seq;  // row of the K and V maps
+    const int q_row0 = (p.head_major ? h * p.B + b : b * p.Hq + h) * p.Sq + q0;               // row of the Q map
+    const int kv_row0 = (p.head_major ? kvh * p.B + b : b * p.Hkv + kvh) * p.cache_seq;  // row of the K and V maps
 
     auto tile_slot = [&](int j) { return WIN && p.ring_cache ? (kv_beg + j * kTcCols) % p.cache_seq : kv_beg + j * kTcCols; };
 
@@ -292,7 +292,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t t_lane = tmem_base + ((uint32_t)(quad * 32) << 16);
         const int qi = min(q0 + row, p.Sq - 1);  // rows past Sq repeat the last one; they are not stored
         const int bound = p.is_causal ? min(active, past + qi + 1) : active;
-        const int first = WIN && p.window > 0 ? max(0, bound - p.window) : 0;  // this row sees [first, bound)
+        const int first = WIN && bound > 0 ? first_visible(bound - 1, p.window, p.chunk) : 0;  // this row sees [first, bound)
         const bool capped = WIN && p.cap2 > 0.f;
         const float sl2 = capped ? 1.f : p.scale * 1.4426950408889634f;  // capped scores are already in log2 units
         float m_used = -INFINITY, l = 0.f;
@@ -318,7 +318,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 for (int i = 0; i < HC; i++)
                     if (col0 + i >= bound) s[i] = -INFINITY;
             }
-            if (WIN && col0 < first) {  // and the tiles at the window's far edge
+            if (WIN && col0 < first) {  // and the tiles at the far edge of the window or chunk
 #pragma unroll
                 for (int i = 0; i < HC; i++)
                     if (col0 + i < first) s[i] = -INFINITY;
@@ -505,9 +505,9 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
     const int last_row = min(q0 + kTcRows, p.Sq) - 1;
     const int kv_end = p.is_causal ? max(0, min(active, past + last_row + 1)) : active;
     // WIN: the walk starts at the tile of the first position that the CTA's first row sees
-    const int kv_beg = WIN ? max(p.window > 0 ? past + q0 + 1 - p.window : 0, max(0, p.ring_cache ? active - p.cache_seq : 0)) / kTcCols * kTcCols : 0;
+    const int kv_beg = WIN ? max(first_visible(max(past + q0, 0), p.window, p.chunk), max(0, p.ring_cache ? active - p.cache_seq : 0)) / kTcCols * kTcCols : 0;
     const int n_tiles = max(0, kv_end - kv_beg + kTcCols - 1) / kTcCols;
-    const int kv_row0 = (b * p.Hkv + kvh) * p.cache_seq;
+    const int kv_row0 = (p.head_major ? kvh * p.B + b : b * p.Hkv + kvh) * p.cache_seq;
 
     auto tile_slot = [&](int j) { return WIN && p.ring_cache ? (kv_beg + j * kTcCols) % p.cache_seq : kv_beg + j * kTcCols; };
 
@@ -546,7 +546,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
             mbar_expect_tx(&q_full, 2 * kTile);
             for (int t = 0; t < 2; t++)
                 for (int sl = 0; sl < SL; sl++)
-                    tma_load_2d(s_q + t * kTile + sl * kTcSlab, &map_q, sl * 128, (b * p.Hq + h0 + t) * p.Sq + q0, &q_full);
+                    tma_load_2d(s_q + t * kTile + sl * kTcSlab, &map_q, sl * 128, (p.head_major ? (h0 + t) * p.B + b : b * p.Hq + h0 + t) * p.Sq + q0, &q_full);
             // a K buffer is free once both heads' S products have read it, a V buffer once both O products have; the loads are
             // issued in the order in which the MMA warp releases the buffers (K0, K1, V0, K2, V1, K3, V2, ...)
             auto load = [&](int j, uint8_t *base, const CUtensorMap *map, uint64_t *full, uint64_t *empty) {
@@ -625,7 +625,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
         const uint32_t colS = t * 128, colO = 256 + t * 128;
         const int qi = min(q0 + row, p.Sq - 1);  // rows past Sq repeat the last one; they are not stored
         const int bound = p.is_causal ? min(active, past + qi + 1) : active;
-        const int first = WIN && p.window > 0 ? max(0, bound - p.window) : 0;  // this row sees [first, bound)
+        const int first = WIN && bound > 0 ? first_visible(bound - 1, p.window, p.chunk) : 0;  // this row sees [first, bound)
         const bool capped = WIN && p.cap2 > 0.f;
         const float sl2 = capped ? 1.f : p.scale * 1.4426950408889634f;  // capped scores are already in log2 units
         float m_used = -INFINITY, l = 0.f;
@@ -648,7 +648,7 @@ attention_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 for (int i = 0; i < kTcCols; i++)
                     if (kv0 + i >= bound) s[i] = -INFINITY;
             }
-            if (WIN && kv0 < first) {  // and the tiles at the window's far edge
+            if (WIN && kv0 < first) {  // and the tiles at the far edge of the window or chunk
 #pragma unroll
                 for (int i = 0; i < kTcCols; i++)
                     if (kv0 + i < first) s[i] = -INFINITY;
@@ -855,7 +855,7 @@ int launch_attention_prefill_tc(cudaStream_t st, void *out, const void *q, const
 bool window_attention_prefill_supported(int dtype, const WindowAttention &w) {
     if (g_prefill_attention_mode <= 0 || !tensor_map_api_available()) return false;
     const bool aligned = (((uintptr_t)w.q | (uintptr_t)w.k | (uintptr_t)w.v | (uintptr_t)w.out) % 16) == 0;
-    return w.Sq >= 16 && w.D == w.E && (w.D == 64 || w.D == 128) && (dtype == MYNN_BF16 || dtype == MYNN_F16) && aligned && w.scale > 0.f &&
+    return w.Sq >= 16 && w.layout != kByToken && w.D == w.E && (w.D == 64 || w.D == 128) && (dtype == MYNN_BF16 || dtype == MYNN_F16) && aligned && w.scale > 0.f &&
            w.cache_rows % kTcCols == 0 && (long long)w.B * w.Hq * w.Sq >= kTcRows && (long long)w.B * w.Hq * w.Sq < (1LL << 31) &&
            (long long)w.B * w.Hkv * w.cache_rows < (1LL << 31);
 }
@@ -874,6 +874,8 @@ int launch_window_attention_prefill(cudaStream_t st, int dtype, const WindowAtte
     p.is_causal = 1;
     p.out_bshd = 1;
     p.window = w.window;
+    p.chunk = w.chunk;
+    p.head_major = w.layout == kByHead;
     p.ring_cache = 1;
     if (w.softcap > 0.f) {
         const float log2e = 1.4426950408889634f;

@@ -1,4 +1,4 @@
-// Causal attention with a sliding window and a score soft cap over ring caches (position p lives in cache row p % cache_rows).
+// Causal attention with a sliding window or chunks and a score soft cap over ring caches (position p lives in cache row p % cache_rows).
 //
 // launch_window_attention picks the kernel: the TMA-ring decode kernel (attention.cu) and the tcgen05 prefill kernels
 // (attention_prefill_tc.cu) take 16-bit tensors with equal key and value sizes of 64 or 128; this file's own kernel takes any
@@ -27,12 +27,14 @@ __global__ void __launch_bounds__(kWinWarps * 32) window_attention_kernel(const 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int active = p.active ? *p.active : p.active_host;
     const int pos = active - p.Sq + sq_i, end = pos + 1;
-    const int lo = max(max(0, active - p.cache_rows), p.window > 0 ? end - p.window : 0);
-    const T *q = reinterpret_cast<const T *>(p.q) + (size_t)blockIdx.x * p.D;
+    const int lo = max(max(0, active - p.cache_rows), first_visible(pos, p.window, p.chunk));
+    const size_t q_row = p.layout == kByBatch ? blockIdx.x : p.layout == kByHead ? ((size_t)h * p.B + b) * p.Sq + sq_i : ((size_t)b * p.Sq + sq_i) * p.Hq + h;
+    const T *q = reinterpret_cast<const T *>(p.q) + q_row * p.D;
     for (int d = threadIdx.x; d < p.D; d += blockDim.x) sq[d] = to_f32<T>(q[d]);
     __syncthreads();
-    const T *kb = reinterpret_cast<const T *>(p.k) + (size_t)(b * p.Hkv + kvh) * p.cache_rows * p.D;
-    const T *vb = reinterpret_cast<const T *>(p.v) + (size_t)(b * p.Hkv + kvh) * p.cache_rows * p.E;
+    const size_t pair = p.layout == kByHead ? (size_t)kvh * p.B + b : (size_t)b * p.Hkv + kvh;
+    const T *kb = reinterpret_cast<const T *>(p.k) + pair * p.cache_rows * p.D;
+    const T *vb = reinterpret_cast<const T *>(p.v) + pair * p.cache_rows * p.E;
     float o[NE], m = -INFINITY, l = 0.f;
 #pragma unroll
     for (int e = 0; e < NE; e++) o[e] = 0.f;
@@ -109,14 +111,15 @@ static int run_window(cudaStream_t st, const WindowAttention &p) {
     else if (p.E <= 64) window_attention_kernel<T, 2><<<rows, kWinWarps * 32, smem, st>>>(p);
     else if (p.E <= 128) window_attention_kernel<T, 4><<<rows, kWinWarps * 32, smem, st>>>(p);
     else if (p.E <= 256) window_attention_kernel<T, 8><<<rows, kWinWarps * 32, smem, st>>>(p);
-    else window_attention_kernel<T, 16><<<rows, kWinWarps * 32, smem, st>>>(p);
+    else if (p.E <= 512) window_attention_kernel<T, 16><<<rows, kWinWarps * 32, smem, st>>>(p);
+    else window_attention_kernel<T, 32><<<rows, kWinWarps * 32, smem, st>>>(p);
     MYNN_LAUNCH_OK("window_attention_kernel");
     return MYNN_OK;
 }
 
 static int check(int dtype, const WindowAttention &p) {
     if (p.B <= 0 || p.Hq <= 0 || p.Hkv <= 0 || p.Sq <= 0 || p.D <= 0 || p.E <= 0 || p.cache_rows <= 0 || p.Hq % p.Hkv) return fail(MYNN_E_ARG, "window_attention: bad shape");
-    if (p.D > 1024 || p.E > 512) return fail(MYNN_E_UNSUPPORTED, "window_attention: head sizes %d / %d", p.D, p.E);
+    if (p.D > 1024 || p.E > 1024 || p.window < 0 || p.chunk < 0) return fail(MYNN_E_UNSUPPORTED, "window_attention: head sizes %d / %d", p.D, p.E);
     if (!dtype_ok(dtype)) return fail(MYNN_E_ARG, "window_attention: bad dtype %d", dtype);
     if (p.Sq > p.cache_rows) return fail(MYNN_E_ARG, "window_attention: %d query rows over a ring of %d rows", p.Sq, p.cache_rows);
     if (!p.out || !p.q || !p.k || !p.v) return fail(MYNN_E_ARG, "window_attention: null pointer");
@@ -140,15 +143,17 @@ int launch_window_attention(cudaStream_t st, int dtype, const WindowAttention &p
 
 using namespace mynn;
 
-extern "C" int mynn_b200_window_attention(void *stream, void *out, const void *q, const void *k, const void *v, float scale, float softcap,
-                                          int window, int B, int Hq, int Hkv, int Sq, int D, int E, int cache_rows, int active,
+extern "C" int mynn_b200_chunk_attention(void *stream, void *out, const void *q, const void *k, const void *v, float scale, float softcap,
+                                         int window, int chunk, int head_major, int B, int Hq, int Hkv, int Sq, int D, int E, int cache_rows, int active,
                                           const int32_t *active_dev, int dtype, void *workspace, size_t workspace_bytes, int plain) {
     WindowAttention p;
     p.out = out;
     p.q = q, p.k = k, p.v = v;
     p.scale = scale;
     p.softcap = softcap;
-    p.window = window;
+    p.window = window > 0 ? window : 0;
+    p.chunk = chunk > 0 ? chunk : 0;
+    p.layout = head_major ? kByHead : kByBatch;
     p.B = B, p.Hq = Hq, p.Hkv = Hkv, p.Sq = Sq, p.D = D, p.E = E;
     p.cache_rows = cache_rows;
     p.active_host = active;
@@ -157,4 +162,11 @@ extern "C" int mynn_b200_window_attention(void *stream, void *out, const void *q
     p.workspace_bytes = workspace_bytes;
     if (!active_dev && (active < Sq || active < 0)) return fail(MYNN_E_ARG, "window_attention: %d positions for %d query rows", active, Sq);
     return plain ? launch_window_attention_plain((cudaStream_t)stream, dtype, p) : launch_window_attention((cudaStream_t)stream, dtype, p);
+}
+
+extern "C" int mynn_b200_window_attention(void *stream, void *out, const void *q, const void *k, const void *v, float scale, float softcap,
+                                          int window, int B, int Hq, int Hkv, int Sq, int D, int E, int cache_rows, int active,
+                                          const int32_t *active_dev, int dtype, void *workspace, size_t workspace_bytes, int plain) {
+    return mynn_b200_chunk_attention(stream, out, q, k, v, scale, softcap, window, 0, 0, B, Hq, Hkv, Sq, D, E, cache_rows, active, active_dev, dtype, workspace,
+                                     workspace_bytes, plain);
 }

@@ -24,7 +24,21 @@ struct GemmView {  // device-side view of DenseGemm
     int M, N, K;
     const int32_t *off, *active, *n_active, *tok_of;  // null: dense
     int gather;
+    int lda, ldo, n_main, act_fn, out_block, batch;
+    long long act_stride, out_stride, out_block_stride;
+    float *out_f32;
 };
+
+// output (row, n) of product z
+template <typename O>
+__device__ __forceinline__ void put_out(const GemmView &g, int z, size_t row, int n, float v) {
+    if (n >= g.n_main) {
+        g.out_f32[row * (g.N - g.n_main) + (n - g.n_main)] = v;
+        return;
+    }
+    const size_t col = g.out_block ? (size_t)(n / g.out_block) * g.out_block_stride + n % g.out_block : n;
+    reinterpret_cast<O *>(g.out)[z * g.out_stride + row * g.ldo + col] = from_f32<O>(dense_act(v, g.act_fn));
+}
 
 // rows [r0, r0 + cnt) of the product and the weight block of group z; false: nothing to do
 __device__ __forceinline__ bool group_rows(const GemmView &g, int z, int &e, int &r0, int &cnt) {
@@ -51,13 +65,14 @@ __global__ void __launch_bounds__(256) dense_tile_kernel(const GemmView g) {
     if (!group_rows(g, blockIdx.z, e, r0, cnt)) return;
     const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
     if (m0 >= cnt) return;
-    const T *act = reinterpret_cast<const T *>(g.act), *w = reinterpret_cast<const T *>(g.w) + (size_t)e * (GLU ? 2 : 1) * g.N * g.K;
+    const int z = g.batch > 1 ? blockIdx.z : 0;
+    const T *act = reinterpret_cast<const T *>(g.act) + z * g.act_stride, *w = reinterpret_cast<const T *>(g.w) + (size_t)(e + z) * (GLU ? 2 : 1) * g.N * g.K;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     float acc[4][4] = {}, accu[GLU ? 4 : 1][4] = {};
     const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;  // loader: row 0..63, four k
     const int am = m0 + lr;
     const T *arow = nullptr;
-    if (am < cnt) arow = act + (size_t)(g.gather ? g.tok_of[r0 + am] : r0 + am) * g.K;
+    if (am < cnt) arow = act + (size_t)(g.gather ? g.tok_of[r0 + am] : r0 + am) * g.lda;
     const T *wrow = n0 + lr < g.N ? w + (size_t)(n0 + lr) * g.K : nullptr;
     const T *urow = GLU && wrow ? wrow + (size_t)g.N * g.K : nullptr;
     for (int k0 = 0; k0 < g.K; k0 += BK) {
@@ -100,7 +115,7 @@ __global__ void __launch_bounds__(256) dense_tile_kernel(const GemmView g) {
             if (n >= g.N) break;
             float v = acc[i][j];
             if constexpr (GLU) v = silu_f(v) * accu[i][j];
-            reinterpret_cast<O *>(g.out)[(size_t)(r0 + m) * g.N + n] = from_f32<O>(v);
+            put_out<O>(g, z, (size_t)(r0 + m), n, v);
         }
     }
 }
@@ -117,12 +132,12 @@ __global__ void __launch_bounds__(kStreamWarps * 32, MT * RT * (GLU ? 2 : 1) <= 
     __shared__ float red[kStreamWarps][WT * 16][MT * 8 + 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, t = lane & 3;
     pdl_trigger();
-    const int n0 = blockIdx.x * 16 * (GLU ? 1 : RT);
+    const int n0 = blockIdx.x * 16 * (GLU ? 1 : RT), z = g.batch > 1 ? blockIdx.y : 0;
     if (!g.off && gridDim.x <= kPrefetchCtas) {
         // launched as a programmatic dependent: the weights of this CTA travel to L2 while the kernel in front of it still runs
         // (a CTA of a later wave starts long after that, for it the prefetch would only be one more request)
         const size_t line = 128 / sizeof(T), total = (size_t)min(16 * (GLU ? 1 : RT), g.N - n0) * g.K;
-        const T *w0 = reinterpret_cast<const T *>(g.w) + (size_t)n0 * g.K;
+        const T *w0 = reinterpret_cast<const T *>(g.w) + ((size_t)z * g.N + n0) * g.K;
         for (size_t i = threadIdx.x * line; i < total; i += kStreamWarps * 32 * line) {
             asm volatile("prefetch.global.L2 [%0];" ::"l"(w0 + i));
             if constexpr (GLU) asm volatile("prefetch.global.L2 [%0];" ::"l"(w0 + (size_t)g.N * g.K + i));
@@ -131,7 +146,7 @@ __global__ void __launch_bounds__(kStreamWarps * 32, MT * RT * (GLU ? 2 : 1) <= 
     pdl_wait();
     int e, r0, cnt;
     if (!group_rows(g, blockIdx.y, e, r0, cnt)) return;
-    const T *act = reinterpret_cast<const T *>(g.act), *w = reinterpret_cast<const T *>(g.w) + (size_t)e * (GLU ? 2 : 1) * g.N * g.K;
+    const T *act = reinterpret_cast<const T *>(g.act) + z * g.act_stride, *w = reinterpret_cast<const T *>(g.w) + (size_t)(e + z) * (GLU ? 2 : 1) * g.N * g.K;
     const T *wp[WT][2];  // this lane's two rows of every tile; rows past N repeat the last one and are not stored
 #pragma unroll
     for (int i = 0; i < WT; i++)
@@ -147,7 +162,7 @@ __global__ void __launch_bounds__(kStreamWarps * 32, MT * RT * (GLU ? 2 : 1) <= 
 #pragma unroll
         for (int i = 0; i < MT; i++) {
             const int m = min(m0 + 8 * i + gq, cnt - 1);
-            ap[i] = act + (size_t)(g.gather ? g.tok_of[r0 + m] : r0 + m) * g.K + 8 * t;
+            ap[i] = act + (size_t)(g.gather ? g.tok_of[r0 + m] : r0 + m) * g.lda + 8 * t;
         }
         float acc[WT][MT][4];
 #pragma unroll
@@ -201,7 +216,7 @@ __global__ void __launch_bounds__(kStreamWarps * 32, MT * RT * (GLU ? 2 : 1) <= 
                     for (int x = 0; x < kStreamWarps; x++) up += red[x][16 + r][m];
                     v = silu_f(v) * up;
                 }
-                reinterpret_cast<O *>(g.out)[(size_t)(r0 + m0 + m) * g.N + n] = from_f32<O>(v);
+                put_out<O>(g, z, (size_t)(r0 + m0 + m), n, v);
             }
         }
         __syncthreads();
@@ -248,8 +263,23 @@ int launch_dense_gemm(cudaStream_t st, int dtype, const DenseGemm &g) {
     if (!dtype_ok(dtype) || (g.out_dtype != dtype && g.out_dtype != MYNN_F32)) return fail(MYNN_E_ARG, "dense_matmul: bad dtypes %d -> %d", dtype, g.out_dtype);
     if (g.M == 0) return MYNN_OK;
     if (!g.out || !g.act || !g.w) return fail(MYNN_E_ARG, "dense_matmul: null pointer");
-    GemmView v = {g.out, g.act, g.w, g.M, g.N, g.K, nullptr, nullptr, nullptr, nullptr, 0};
-    int groups = 1;
+    if (g.out_f32 ? g.n_main <= 0 || g.n_main > g.N : g.n_main != 0) return fail(MYNN_E_ARG, "dense_matmul: %d of %d columns in the main output", g.n_main, g.N);
+    if (g.batch < 1 || g.batch > 65535 || (g.batch > 1 && (g.route || g.out_f32)) || (g.route && (g.out_f32 || g.out_block || g.lda || g.ldo)) ||
+        (g.glu && (g.act_fn || g.out_f32)) || g.out_block < 0)
+        return fail(MYNN_E_ARG, "dense_matmul: options that do not go together");
+    GemmView v = {};
+    v.out = g.out, v.act = g.act, v.w = g.w;
+    v.M = g.M, v.N = g.N, v.K = g.K;
+    v.n_main = g.out_f32 ? g.n_main : g.N;
+    v.lda = g.lda ? g.lda : g.K;
+    v.ldo = g.ldo ? g.ldo : v.n_main;
+    v.act_fn = g.act_fn;
+    v.out_block = g.out_block;
+    v.out_block_stride = g.out_block_stride;
+    v.batch = g.batch;
+    v.act_stride = g.act_stride, v.out_stride = g.out_stride;
+    v.out_f32 = g.out_f32;
+    int groups = g.batch;
     long long rows = g.M;  // rows a weight block meets on average
     if (g.route) {
         v.off = g.route->off;
@@ -262,9 +292,9 @@ int launch_dense_gemm(cudaStream_t st, int dtype, const DenseGemm &g) {
         rows = (pairs + g.experts - 1) / g.experts * 2;  // the fuller experts of an uneven choice
         if (rows > g.M) rows = g.M;
     }
-    const bool aligned = (((uintptr_t)g.act | (uintptr_t)g.w) % 16) == 0 && g.K % 8 == 0 && dtype != MYNN_F32;
+    const bool aligned = (((uintptr_t)g.act | (uintptr_t)g.w) % 16) == 0 && g.K % 8 == 0 && v.lda % 8 == 0 && g.act_stride % 8 == 0 && dtype != MYNN_F32;
     if (dense_gemm_tc_supported(dtype, g)) return launch_dense_gemm_tc(st, dtype, g);
-    const bool stream = aligned && rows <= 64;
+    const bool stream = aligned && (rows <= 64 || g.batch > 1);
     const bool f32out = g.out_dtype == MYNN_F32;
     if (dtype == MYNN_F32) return run_tile<float, float>(st, v, groups, g.glu);
     if (dtype == MYNN_BF16) {
@@ -288,6 +318,27 @@ extern "C" int mynn_b200_dense_matmul(void *stream, void *out, const void *act, 
     g.M = M, g.N = N, g.K = K;
     g.out_dtype = out_dtype;
     g.glu = glu;
+    g.status = status;
+    return launch_dense_gemm((cudaStream_t)stream, dtype, g);
+}
+
+extern "C" int mynn_b200_dense_matmul_ex(void *stream, void *out, const void *act, const void *w, int M, int N, int K, int dtype, int out_dtype, int act_fn,
+                                         float *out_f32, int n_main, int out_block, long long out_block_stride, int lda, int ldo, int batch,
+                                         long long act_stride, long long out_stride, int32_t *status) {
+    DenseGemm g;
+    g.out = out;
+    g.act = act;
+    g.w = w;
+    g.M = M, g.N = N, g.K = K;
+    g.out_dtype = out_dtype;
+    g.act_fn = act_fn;
+    g.out_f32 = out_f32;
+    g.n_main = n_main;
+    g.out_block = out_block;
+    g.out_block_stride = out_block_stride;
+    g.lda = lda, g.ldo = ldo;
+    g.batch = batch;
+    g.act_stride = act_stride, g.out_stride = out_stride;
     g.status = status;
     return launch_dense_gemm((cudaStream_t)stream, dtype, g);
 }

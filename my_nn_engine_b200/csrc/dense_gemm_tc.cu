@@ -34,6 +34,9 @@ struct DgParams {
     int n_tiles;                                  // weight tiles
     const int32_t *off, *tile_e, *tile_row, *m_tiles_dev;  // grouped: see MoeRoute; null: dense
     int row_fastest;                              // dense: walk the row tiles fastest
+    int ldo, n_main, act_fn, out_block;           // see DenseGemm; out_block 0: none
+    long long out_block_stride;
+    float *out_f32;
     int *status;
 };
 
@@ -173,7 +176,9 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
     } else {
         // ---------------- epilogue warps 2..5: lane quadrant = warp & 3, one activation row per thread ----------------
         const int quad = warp & 3, row = quad * 32 + lane;
-        const bool vec = p.N % (sizeof(O) == 4 ? 4 : 8) == 0 && (uintptr_t)p.out % 16 == 0;
+        constexpr int kPiece = sizeof(O) == 4 ? 4 : 8;  // elements of a 16-byte store
+        const bool vec = p.ldo % kPiece == 0 && (uintptr_t)p.out % 16 == 0 && p.out_block % kPiece == 0 && p.out_block_stride % kPiece == 0;
+        const bool runs = p.out_block % 32 == 0;        // 32 neighbouring columns from a multiple of 32 on lie in one block
         int it = 0;
         for (int tile = blockIdx.x; tile < total; tile += gridDim.x, it++) {
             const int buf = it & 1, use = it >> 1;
@@ -193,7 +198,8 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
             const uint32_t t_lane = tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(buf * kDgCols);
             const int n0 = nt * NT;
             const bool mine = r0 + row < end;
-            O *out = reinterpret_cast<O *>(p.out) + (size_t)(r0 + row) * p.N + n0;
+            O *out = reinterpret_cast<O *>(p.out) + (size_t)(r0 + row) * p.ldo;
+            float *out_f32 = p.out_f32 + (size_t)(r0 + row) * (p.N - p.n_main);  // not read without out_f32
 #pragma unroll 1
             for (int c = 0; c < NT; c += 32) {
                 if (n0 + c >= p.N) break;  // uniform
@@ -208,7 +214,24 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
                 } else {
                     tmem_ld_wait();
                 }
-                if (mine) store_run<T, O>(out + c, v, min(32, p.N - n0 - c), vec);
+                if (mine) {
+                    const int n = n0 + c, run = min(32, p.N - n);
+                    if (n + run <= p.n_main && runs) {
+                        if (p.act_fn) {
+#pragma unroll
+                            for (int i = 0; i < 32; i++) v[i] = dense_act(v[i], p.act_fn);
+                        }
+                        store_run<T, O>(out + (p.out_block ? (size_t)(n / p.out_block) * p.out_block_stride + n % p.out_block : (size_t)n), v, run, vec);
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 32; i++) {
+                            if (i >= run) continue;
+                            const int j = n + i;
+                            if (j >= p.n_main) out_f32[j - p.n_main] = v[i];
+                            else out[p.out_block ? (size_t)(j / p.out_block) * p.out_block_stride + j % p.out_block : (size_t)j] = from_f32<O>(dense_act(v[i], p.act_fn));
+                        }
+                    }
+                }
             }
             tc_fence_before();
             __syncwarp();
@@ -229,7 +252,7 @@ __global__ void __launch_bounds__(256) gather_places_kernel(uint4 *out, const ui
 }
 
 bool dense_gemm_tc_supported(int dtype, const DenseGemm &g) {
-    if (dtype == MYNN_F32 || !g.status || !tensor_map_api_available() || g.K % 8 || (((uintptr_t)g.act | (uintptr_t)g.w) % 16)) return false;
+    if (dtype == MYNN_F32 || !g.status || !tensor_map_api_available() || g.K % 8 || g.batch > 1 || (g.lda && g.lda != g.K) || (((uintptr_t)g.act | (uintptr_t)g.w) % 16)) return false;
     const long long wrows = (long long)g.experts * g.N * (g.glu ? 2 : 1), arows = g.route ? (long long)g.M * g.top : g.M;
     if (wrows >= (1ll << 31) || arows >= (1ll << 31)) return false;
     if (!g.route) return g.M > 32;
@@ -274,6 +297,12 @@ int launch_dense_gemm_tc(cudaStream_t st, int dtype, const DenseGemm &g) {
     const int nt = g.glu ? kDgCols / 2 : kDgCols;
     p.n_tiles = (g.N + nt - 1) / nt;
     p.status = g.status;
+    p.n_main = g.out_f32 ? g.n_main : g.N;
+    p.ldo = g.ldo ? g.ldo : p.n_main;
+    p.act_fn = g.act_fn;
+    p.out_block = g.out_block;
+    p.out_block_stride = g.out_block_stride;
+    p.out_f32 = g.out_f32;
     long long m_bound = (g.M + kDgRows - 1) / kDgRows;
     if (g.route) {
         p.off = g.route->off;

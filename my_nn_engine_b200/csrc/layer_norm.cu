@@ -1,4 +1,4 @@
-// Layer norms of the block decoder, fused with the residual step in front of them.
+// Layer norms (and norms by root mean square) of the block decoder, fused with the residual step in front of them.
 //
 // A sandwich-normed layer does x += mult * LN(sublayer output) and then feeds LN(x) to the next sublayer.  Both norms, the
 // residual sum, the combination of routed experts and the addition of the embedding output at the start of a repeated pass
@@ -106,6 +106,15 @@ __global__ void __launch_bounds__(NV == 1 ? 256 : 1024) norm_step_kernel(const N
             }
         return block_moments(m, sm);
     };
+    // reciprocal deviation; for a norm by root mean square nothing is taken off, and mean(v^2) = var + mean^2
+    auto scale_of = [&](Moments &m) {
+        float v = m.m2 / (float)W;
+        if (p.rms) {
+            v += m.mean * m.mean;
+            m.mean = 0.f;
+        }
+        return 1.0f / sqrtf(v + p.eps);
+    };
     if (p.embed) {
         const long long id = min(max((long long)p.ids[row], 0ll), (long long)p.vocab - 1);
         const T *e = reinterpret_cast<const T *>(p.embed) + (size_t)id * W;
@@ -155,15 +164,21 @@ __global__ void __launch_bounds__(NV == 1 ? 256 : 1024) norm_step_kernel(const N
                     if (i < W) load_vec<T, V>(sub + (size_t)row * W + i, sv[j]);
                 }
             }
-            const Moments m = moments(sv);
-            const float inv = 1.0f / sqrtf(m.m2 / (float)W + p.eps);
+            Moments m = {0.f, 0.f, 0.f};
+            float inv = 1.f;
+            if (p.w1) {
+                m = moments(sv);
+                inv = scale_of(m);
+            }
 #pragma unroll
             for (int j = 0; j < NV; j++) {
                 const int i = i0 + j * step;
                 if (i < W) {
                     float w[V], b[V], z[V];
-                    load_vec<float, V>(p.w1 + i, w);
-                    load_vec<float, V>(p.b1 + i, b);
+#pragma unroll
+                    for (int k = 0; k < V; k++) w[k] = 1.f, b[k] = 0.f;
+                    if (p.w1) load_vec<float, V>(p.w1 + i, w);
+                    if (p.w1 && !p.rms) load_vec<float, V>(p.b1 + i, b);
                     if (p.add_x0) load_vec<float, V>(p.x0 + (size_t)row * W + i, z);
 #pragma unroll
                     for (int k = 0; k < V; k++) {
@@ -176,8 +191,8 @@ __global__ void __launch_bounds__(NV == 1 ? 256 : 1024) norm_step_kernel(const N
         }
     }
     if (!p.out) return;
-    const Moments m = moments(xv);
-    const float inv = 1.0f / sqrtf(m.m2 / (float)W + p.eps);
+    Moments m = moments(xv);
+    const float inv = scale_of(m);
     T *out = reinterpret_cast<T *>(p.out) + (size_t)row * W;
 #pragma unroll
     for (int j = 0; j < NV; j++) {
@@ -185,7 +200,9 @@ __global__ void __launch_bounds__(NV == 1 ? 256 : 1024) norm_step_kernel(const N
         if (i < W) {
             float w[V], b[V], y[V];
             load_vec<float, V>(p.w2 + i, w);
-            load_vec<float, V>(p.b2 + i, b);
+#pragma unroll
+            for (int k = 0; k < V; k++) b[k] = 0.f;
+            if (!p.rms) load_vec<float, V>(p.b2 + i, b);
 #pragma unroll
             for (int k = 0; k < V; k++) y[k] = (xv[j][k] - m.mean) * inv * w[k] + b[k];
             store_vec<T, V>(out + i, y);
@@ -260,6 +277,22 @@ extern "C" int mynn_b200_residual_layer_norm(void *stream, float *x, const void 
     p.b2 = bias;
     p.mult = mult;
     p.eps = eps;
+    p.out = out;
+    p.W = W;
+    return launch_norm_step((cudaStream_t)stream, dtype, p, rows);
+}
+
+extern "C" int mynn_b200_residual_rms_norm(void *stream, float *x, const void *sub, const float *weight, void *out, float eps, int rows, int W, int dtype) {
+    if (rows < 0 || W <= 0) return fail(MYNN_E_ARG, "residual_rms_norm: bad shape rows=%d W=%d", rows, W);
+    if (!dtype_ok(dtype)) return fail(MYNN_E_ARG, "residual_rms_norm: bad dtype %d", dtype);
+    if (rows == 0) return MYNN_OK;
+    if (!x || (out && !weight)) return fail(MYNN_E_ARG, "residual_rms_norm: null pointer");
+    NormStep p;
+    p.x = x;
+    p.sub = sub;
+    p.w2 = weight;
+    p.eps = eps;
+    p.rms = 1;
     p.out = out;
     p.W = W;
     return launch_norm_step((cudaStream_t)stream, dtype, p, rows);

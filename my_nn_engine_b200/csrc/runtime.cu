@@ -44,7 +44,7 @@ extern "C" const char *mynn_b200_last_error(void) {
     return copy;
 }
 
-extern "C" int mynn_b200_abi_version(void) { return 1; }
+extern "C" int mynn_b200_abi_version(void) { return 2; }
 
 extern "C" int mynn_b200_compiled_arch(void) {
 #ifdef MYNN_COMPILED_ARCH

@@ -72,7 +72,10 @@ class DeviceModel:
     """A model resident on the current CUDA device behind the library's model entry points: what every model family shares.
 
     A subclass lays out its weights and state buffers and calls ``_open`` with its configuration; steps, prefill chunks and
-    their host staging are the same for all."""
+    their host staging are the same for all.  ``can_rewind``: a step may go back behind the last position stored (a model with
+    recurrent state cannot)."""
+
+    can_rewind = True
 
     def _open(self, configure, config, init, states, logits_dtype):
         """configure + model_init, then the pinned host staging."""

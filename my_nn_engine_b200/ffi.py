@@ -14,6 +14,8 @@ LIB_PATH = os.path.join(HERE, "libmynn_b200.so")
 
 F32, BF16, F16 = 0, 1, 2
 W_NK, W_KN = 0, 1
+MIX_ATTENTION, MIX_LATENT, MIX_MLSTM = 0, 1, 2
+ACT_NONE, ACT_SQUARE_RELU = 0, 1
 OK, E_ARG, E_CUDA, E_UNSUPPORTED, E_COMM, E_STATE = 0, -1, -2, -3, -4, -5
 OPT_WAIT_BUDGET_US, OPT_KSPLIT, OPT_PREFILL_ATTENTION, OPT_INJECT_STALL, OPT_FUSE_ROPE, OPT_DECODE_RING = 1, 2, 3, 4, 5, 6
 
@@ -36,14 +38,15 @@ class Block(ctypes.Structure):
     """Mirror of ``mynn_b200_block``: one layer of a block decoder."""
 
     _fields_ = [(n, c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "conv_taps", "rot_dims", "window", "cache_rows", "history_rows",
-                                       "experts", "expert_ff", "top", "groups", "groups_keep")] + [("attn_scale", c_float), ("softcap", c_float)]
+                                       "experts", "expert_ff", "top", "groups", "groups_keep", "mixer", "rot_halves", "qk_norm", "chunk", "q_rank", "kv_rank",
+                                       "dense_ff", "ff_act")] + [("attn_scale", c_float), ("softcap", c_float), ("gate_cap", c_float)]
 
 
 class BlockModelConfig(ctypes.Structure):
     """Mirror of ``mynn_b200_block_model_config``."""
 
     _fields_ = [(n, c_int32) for n in ("n_layers", "hidden", "vocab", "max_seq_len", "batch", "dtype", "output_mode", "use_graph", "max_prefill",
-                                       "max_rewind", "loop_start", "loop_stop", "loop_times")] + \
+                                       "max_rewind", "loop_start", "loop_stop", "loop_times", "rms_norm", "post_norm")] + \
                [(n, c_float) for n in ("embed_scale", "residual_mult", "norm_eps")] + [("layers", POINTER(Block))]
 
 
@@ -108,6 +111,14 @@ SIGNATURES = {
     "mynn_b200_residual_layer_norm": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_int, c_int, c_int]),
     "mynn_b200_short_conv_append": (c_int, [c_void_p] * 9 + [c_int] * 10 + [c_void_p, c_int]),
     "mynn_b200_window_attention": (c_int, [c_void_p] * 5 + [c_float, c_float] + [c_int] * 9 + [c_void_p, c_int, c_void_p, c_size_t, c_int]),
+    "mynn_b200_chunk_attention": (c_int, [c_void_p] * 5 + [c_float, c_float] + [c_int] * 11 + [c_void_p, c_int, c_void_p, c_size_t, c_int]),
+    "mynn_b200_residual_rms_norm": (c_int, [c_void_p] * 5 + [c_float, c_int, c_int, c_int]),
+    "mynn_b200_rotary_append": (c_int, [c_void_p] * 7 + [c_int] * 9 + [c_float, c_int, c_void_p, c_int]),
+    "mynn_b200_latent_append": (c_int, [c_void_p] * 6 + [c_float] + [c_int] * 5 + [c_void_p, c_int]),
+    "mynn_b200_latent_attention_workspace_bytes": (c_size_t, [c_int] * 5),
+    "mynn_b200_latent_attention": (c_int, [c_void_p] * 4 + [c_float] + [c_int] * 6 + [c_void_p, c_int, c_void_p, c_size_t, c_int]),
+    "mynn_b200_mlstm": (c_int, [c_void_p] * 9 + [c_float, c_float] + [c_int] * 5 + [c_void_p] * 3 + [c_int, c_int]),
+    "mynn_b200_dense_matmul_ex": (c_int, [c_void_p] * 4 + [c_int] * 6 + [c_void_p, c_int, c_int, ctypes.c_longlong, c_int, c_int, c_int, ctypes.c_longlong, ctypes.c_longlong, c_void_p]),
     "mynn_b200_moe_workspace_bytes": (c_size_t, [c_int, c_int, c_int]),
     "mynn_b200_moe_route": (c_int, [c_void_p, c_void_p, c_size_t, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int]),
     "mynn_b200_dense_matmul": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),

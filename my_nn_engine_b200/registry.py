@@ -11,7 +11,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable, List
 
-from . import vebisun
+from . import fimadra, vebisun
 from .checkpoint import load_model_dir, load_weights_dir
 from .decoder import DecoderModel
 
@@ -41,7 +41,16 @@ def _build_vebisun(model_dir, cfg, **options):
     return vebisun.build(cfg, load_weights_dir(model_dir), **options)
 
 
-FAMILIES: List[Family] = [Family("llama", _is_llama, _build_llama), Family("vebisun", _is_vebisun, _build_vebisun)]
+def _is_fimadra(cfg: dict) -> bool:
+    return cfg.get("architecture") == fimadra.ARCHITECTURE
+
+
+def _build_fimadra(model_dir, cfg, **options):
+    return fimadra.build(cfg, load_weights_dir(model_dir), **options)
+
+
+FAMILIES: List[Family] = [Family("llama", _is_llama, _build_llama), Family("vebisun", _is_vebisun, _build_vebisun),
+                          Family("fimadra", _is_fimadra, _build_fimadra)]
 
 
 def read_config(model_dir: str) -> dict:

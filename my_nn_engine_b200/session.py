@@ -49,6 +49,7 @@ class LlmSession:
         self.tokenizer = tokenizer
         self._past_len = 0
         self._feed = None
+        self._stored = None    # token of every position the model holds (kept for a model that cannot rewind)
         self.streaming = None  # (sink, window) when bound to a streaming-cache model: the stream has no length limit
 
     @classmethod
@@ -95,7 +96,26 @@ class LlmSession:
         make = cls.for_llama_streaming if getattr(model, "streaming", None) else cls.for_llama
         self = make(model, eos_token_id, prefill_len, tokenizer)
         self._feed = getattr(model, "feed", None)
+        if not getattr(model, "can_rewind", True):
+            self._stored = []
         return self
+
+    def _catch_up(self):
+        """A conversation that dropped its last tokens goes on behind them.  Cached rows are simply overwritten; a recurrent state
+        cannot go back, so what is left of the conversation runs again from its beginning."""
+        if self._stored is None or len(self._stored) == self._past_len:
+            return
+        ids, self._stored, self._past_len = self._stored[:self._past_len], [], 0
+        if self.prefill_len:
+            self._run_prefill(ids)
+        else:
+            for t in ids:
+                self._step(t)
+
+    def _advance(self, tokens):
+        self._past_len += len(tokens)
+        if self._stored is not None:
+            self._stored += tokens
 
     def feed(self, tokens: Sequence[int], want: Sequence[int] = ()):
         """Append given tokens to the sequence without picking any: prefill chunks and decode steps at the current past_len.
@@ -104,8 +124,9 @@ class LlmSession:
             raise ValueError("feed() needs a model bound with for_model() and a plain cache")
         if self.max_seq_len < self._past_len + len(tokens):
             raise PromptTooLong(self._past_len + len(tokens), self.max_seq_len, self._past_len)
+        self._catch_up()
         out = self._feed(tokens, self._past_len, want)
-        self._past_len += len(tokens)
+        self._advance(list(tokens))
         return out
 
     def past_len(self) -> int:
@@ -115,6 +136,8 @@ class LlmSession:
         """Forget the conversation: only ``past_len`` is zeroed, the cache rows are simply overwritten later
         (crates/llm/src/session.rs:303-305)."""
         self._past_len = 0
+        if self._stored is not None:
+            self._stored = []
 
     def _encode(self, prompt):
         if isinstance(prompt, str):
@@ -147,13 +170,13 @@ class LlmSession:
             else:
                 chunk = prompt_ids[pos:pos + 1]
                 tok = self._decode_step(chunk[0], self._past_len)
-            self._past_len += len(chunk)
+            self._advance(chunk)
             pos += len(chunk)
         return tok
 
     def _step(self, token):
         nxt = self._decode_step(token, self._past_len)
-        self._past_len += 1
+        self._advance([token])
         return nxt
 
     def generate_ids(self, prompt, max_new_tokens: int = 16, opts: Optional[GenerateOptions] = None,
@@ -174,6 +197,7 @@ class LlmSession:
             if not self.streaming and self.max_seq_len < self._past_len + 1:
                 break
             if i == 0:
+                self._catch_up()
                 if self.prefill_len:
                     token = self._run_prefill(prompt_ids)
                 else:

@@ -28,7 +28,7 @@ def test_header_symbols_are_exported_and_bound():
 
 
 def test_version_and_arch():
-    assert ffi.lib().mynn_b200_abi_version() == 1
+    assert ffi.lib().mynn_b200_abi_version() == 2
     assert ffi.lib().mynn_b200_compiled_arch() == 100
 
 
