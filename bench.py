@@ -2,7 +2,7 @@
 batch 32, 2048-token context, greedy decode — tokens per second of the whole job.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
-    python bench.py --case {gemv|gemm|attention|prefill_gemm|prefill_attention|prefill_model|w8a8|suite|block|block_kernels} [...]
+    python bench.py --case {gemv|gemm|attention|prefill_gemm|prefill_attention|prefill_model|w8a8|suite|block|block_kernels|fimadra|fimadra_kernels} [...]
 
 Default case ("step").  A step is one decode step of the whole batch (32 new tokens).  Weights are random-init (N(0, 0.02),
 quantised with the engine's quantizer), the 2048-token context is synthetic KV (N(0,1) * 0.5, one seed for the whole cache,
@@ -24,6 +24,7 @@ The other cases time single kernels of the path the way the step's kernels are f
 its weights / KV (copies x size > L2), the launches are replayed from one CUDA graph, CUDA events on the launching stream.
 block: prefill and decode throughput of Vebisun-shaped models with layers like those of real ones, beside the int8 Llama graph at
 equal width, heads, depth and feed-forward width per token; block_kernels: their kernels one by one against the roofline.
+fimadra / fimadra_kernels: the same for Fimadra-shaped models, beside Vebisun-shaped ones of equal width, heads, depth and feed-forward bytes.
 Algorithmic bytes: GEMM  N*K + N*sizeof(scale) + M*K*sizeof(act) + M*N*sizeof(out);  attention  2*B*Hkv*L*D*2 + Q + out.
 """
 from __future__ import annotations
@@ -777,11 +778,12 @@ def _model_throughput(model, vocab, batch, context, steps=64, chunk=2048):
         for i in range(8):
             model.step_device(ids if i == 0 else None, context + i)
         times = []
-        for _ in range(3):
+        for rep in range(3):  # the same positions again, or further ones where the state cannot go back
+            at = context + 8 + (0 if model.can_rewind else rep * steps)
             e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             e0.record(stream)
             for i in range(steps):
-                model.step_device(None, context + 8 + i)
+                model.step_device(None, at + i)
             e1.record(stream)
             torch.cuda.synchronize()
             times.append(e0.elapsed_time(e1) / steps)
@@ -898,6 +900,189 @@ def case_block_kernels(name, batch, context=2048):
         raise RuntimeError(f"dense_matmul: a bounded wait ran out (status {int(status.item())})")
 
 
+# --------------------------------------------------------------------------------------------------------
+# Fimadra: layers like those of real models, random weights, beside a Vebisun-shaped model at equal size
+# --------------------------------------------------------------------------------------------------------
+# layers run [latent, attention, mlstm, mlstm] over and over; the mlstm layers have no feed-forward
+FIMADRA_ARCHS = {
+    "small": dict(width=2048, heads=16, kv=4, dim=128, chunk=1024, q_rank=768, kv_rank=512, mem_heads=4, mem_dim=256, mem_vdim=512, ff=8192, layers=8, vocab=32000),
+    "large": dict(width=4096, heads=32, kv=8, dim=128, chunk=2048, q_rank=1536, kv_rank=512, mem_heads=8, mem_dim=256, mem_vdim=512, ff=16384, layers=4, vocab=32000),
+}
+
+
+def fimadra_model(a, batch, max_seq, max_prefill):
+    import torch
+
+    from my_nn_engine_b200.block_decoder import BlockDecoder, BlockLayer, BlockModelSpec, Rotary
+    g = torch.Generator(device="cuda").manual_seed(0)
+    W, H, D = a["width"], a["heads"], a["dim"]
+
+    def mat(*shape):
+        return torch.empty(*shape, device="cuda", dtype=torch.bfloat16).normal_(0.0, 0.02, generator=g)
+
+    def ones(n):
+        return torch.ones(n, device="cuda")
+
+    ff = dict(dense_ff=a["ff"], ff_act="square_relu")
+    lat = BlockLayer(mixer="latent_attention", heads=H, kv_heads=H, dim=D, vdim=D, scale=D ** -0.5, q_rank=a["q_rank"], kv_rank=a["kv_rank"], **ff)
+    att = BlockLayer(heads=H, kv_heads=a["kv"], dim=D, vdim=D, scale=D ** -0.5, chunk=a["chunk"], rotary=Rotary(1e6, D), rot_halves=True, qk_norm=True, **ff)
+    mem = BlockLayer(mixer="mlstm", heads=a["mem_heads"], kv_heads=a["mem_heads"], dim=a["mem_dim"], vdim=a["mem_vdim"], scale=1.0, gate_cap=15.0)
+    layers = ([lat, att, mem, mem] * a["layers"])[:a["layers"]]
+    spec = BlockModelSpec(hidden=W, vocab=a["vocab"], layers=layers, norm_eps=1e-6, rms_norm=True, post_norm=False, logit_scale=0.5)
+    weights = {"embed": mat(a["vocab"], W), "head": mat(a["vocab"], W), "final_norm": (ones(W), None), "layers": []}
+    for L in layers:
+        w = {"norm1": (ones(W), None), "norm2": (ones(W), None), "qkv": mat(L.channels, W), "conv": None, "o": mat(W, L.heads * L.vdim)}
+        if L.dense_ff:
+            w.update(up=mat(L.dense_ff, W), down=mat(W, L.dense_ff))
+        if L.mixer == "latent_attention":
+            w.update(q_norm=ones(L.q_rank), kv_norm=ones(L.kv_rank), uq=mat(H * D, L.q_rank), uk=mat(H * D, L.kv_rank), uv=mat(H * D, L.kv_rank))
+        if L.mixer == "mlstm":
+            w.update(head_norm=ones(L.heads * L.vdim), gate_bias=torch.cat([torch.zeros(L.heads), 4.0 * torch.ones(L.heads)]))
+        weights["layers"].append(w)
+    return BlockDecoder(spec, weights, dtype="bf16", max_seq_len=max_seq, batch=batch, output="ids", max_prefill=max_prefill)
+
+
+def vebisun_beside(a, batch, max_seq, max_prefill):
+    """Equal width, heads, depth, vocabulary; one expert whose three matrices are as large as the dense feed-forward's two."""
+    b = dict(width=a["width"], heads=a["heads"], kv=a["kv"], dim=a["dim"], window=a["chunk"], experts=1, top=1, ff=a["ff"] * 2 // 3 // 16 * 16, groups=1, keep=1,
+             layers=a["layers"], vocab=a["vocab"])
+    return block_model(b, batch, max_seq, max_prefill)
+
+
+def case_fimadra(name, batch, context=2048):
+    import torch
+    a = FIMADRA_ARCHS[name]
+    chunk = max(64, 2048 // batch)
+    out = {"case": "fimadra", "arch": name, **a, "batch": batch, "context": context, "chunk_tokens": chunk, "data": "synthetic"}
+    for key, make in (("fimadra_bf16", fimadra_model), ("vebisun_bf16", vebisun_beside)):
+        m = make(a, batch, context + 256, chunk)
+        l0 = m.lib.mynn_b200_launch_count()
+        tps, ms = _model_throughput(m, a["vocab"], batch, context, chunk=chunk)
+        out[key] = {"prefill_tok_per_s": tps, "decode_ms_per_step": ms, "decode_tok_per_s": batch * 1e3 / ms, "weight_bytes": m.weight_bytes(),
+                    "kernels_launched": m.lib.mynn_b200_launch_count() - l0}
+        m.close()
+        del m
+        torch.cuda.empty_cache()
+    return out
+
+
+def case_fimadra_kernels(name, rows, context=2048):
+    """The kernels of the three mixers at a decode step of ``rows`` sequences (rows > 32: at a prefill chunk of that many tokens) against
+    their rooflines (the slower of bytes and operations), each next to the like kernel of a Vebisun-shaped model."""
+    import torch
+
+    from my_nn_engine_b200 import ffi, ops
+    a, M = FIMADRA_ARCHS[name], rows
+    hbm, tf, kind = measured_peaks()
+    W, H, G, D, Q, R, ff, ck = (a[k] for k in ("width", "heads", "kv", "dim", "q_rank", "kv_rank", "ff", "chunk"))
+    MH, MD, ME = a["mem_heads"], a["mem_dim"], a["mem_vdim"]
+    prefill = M > 32
+    B, S = (1, M) if prefill else (M, 1)
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+
+    def rnd(*shape):
+        return torch.empty(*shape, device="cuda", dtype=torch.bfloat16).normal_(0.0, 0.05)
+
+    def figure(what, us, nbytes, flops, like=False):
+        floor = max(nbytes / hbm / 1e3, flops / tf / 1e6)
+        return {"case": "fimadra_kernels", "arch": name, "rows": M, ("like" if like else "kernel"): what, "us": us, "GBps": nbytes / us / 1e3, "TFLOPs": flops / us / 1e6,
+                "bound": "hbm" if nbytes / hbm / 1e3 > flops / tf / 1e6 else "tensor", "frac_of_%s" % kind: floor / us}
+
+    def copies(nbytes):
+        return max(3, int(400e6 // nbytes) + 1)
+
+    def product(what, N, K, like=False, **kw):
+        act, ws = rnd(M, K), [rnd(N, K) for _ in range(copies(2 * N * K))]
+        if kw:
+            fn = lambda w: ops.dense_matmul_ex(act, w, status=status, **kw)  # noqa: E731
+        else:
+            fn = lambda w: ops.dense_matmul(act, w, status=status)  # noqa: E731
+        us = _time_launches([(lambda w=w: fn(w)) for w in ws])
+        return figure(f"{what} {N}x{K}", us, 2 * (N * K + M * K + M * N), 2.0 * M * N * K, like)
+
+    mem_cols = 2 * MH * (MD + ME) + 2 * MH
+    yield product("mlstm product with f32 gates", mem_cols, W, f32_columns=2 * MH)
+    yield product("plain product", mem_cols, W, like=True)
+    yield product("up product with squared relu", ff, W, act_fn=ffi.ACT_SQUARE_RELU)
+    yield product("plain product", ff, W, like=True)
+    yield product("down product", W, ff)
+    yield product("latents", Q + R, W)
+    yield product("latent queries", H * D, Q, **(dict(block=D) if prefill else {}))
+    if prefill:
+        yield product("keys of latents", H * D, R, block=D)
+        yield product("plain product", H * D, R, like=True)
+    else:
+        for what, N, K in (("queries into latent space, per head", R, D), ("values of latents, per head", D, R)):
+            act, ws = rnd(M, H, K), [rnd(H, N, K) for _ in range(copies(2 * H * N * K))]
+            us = _time_launches([(lambda w=w: ops.dense_matmul_heads(act, w)) for w in ws])
+            yield figure(f"{what} {H}x{N}x{K}", us, 2 * H * (N * K + M * K + M * N), 2.0 * M * H * N * K)
+        yield product("plain product of as many weights", H * R, D, like=True)
+        yield product("plain product of as many weights", D, H * R, like=True)
+    # ---- attention ----
+    if prefill:
+        seen = sum(i % ck + 1 for i in range(S))
+        wseen = sum(min(i + 1, ck) for i in range(S))
+        rws = -(-(min(ck - 1, context) + S) // 128) * 128
+        q, k, v = rnd(1, H, S, D), rnd(1, G, rws, D), rnd(1, G, rws, D)
+        us = _time_launches([lambda: ops.chunk_attention(q, k, v, D ** -0.5, S, chunk=ck)] * 4)
+        yield figure(f"chunk attention, {S} tokens, chunks of {ck}", us, 2 * S * D * (2 * H + 2 * G), 4.0 * seen * D * H)
+        us = _time_launches([lambda: ops.window_attention(q, k, v, D ** -0.5, S, ck, 30.0)] * 4)
+        yield figure(f"window attention, {S} tokens, window {ck}, soft cap", us, 2 * S * D * (2 * H + 2 * G), 4.0 * wseen * D * H, like=True)
+        q, k, v = rnd(H, 1, S, D), rnd(H, 1, -(-S // 128) * 128, D), rnd(H, 1, -(-S // 128) * 128, D)
+        us = _time_launches([lambda: ops.chunk_attention(q, k, v, D ** -0.5, S, head_major=True)] * 4)
+        yield figure(f"attention over expanded latents, {S} tokens", us, 8 * S * D * H, 2.0 * S * (S + 1) * D * H)
+    else:
+        n = min(ck, context)
+        rws = -(-(ck + 256) // 128) * 128
+        kv = 2 * M * G * n * D * 2
+        ks, vs = [[rnd(M, G, rws, D) for _ in range(copies(kv // 2))] for _ in range(2)]
+        q = rnd(M, H, 1, D)
+        us = _time_launches([(lambda k=k, v=v: ops.chunk_attention(q, k, v, D ** -0.5, n, chunk=ck)) for k, v in zip(ks, vs)])
+        yield figure(f"chunk attention, decode, {n} rows seen", us, kv + 4 * q.numel(), 4.0 * M * H * n * D)
+        us = _time_launches([(lambda k=k, v=v: ops.window_attention(q, k, v, D ** -0.5, n, ck, 30.0)) for k, v in zip(ks, vs)])
+        yield figure(f"window attention, decode, {n} rows seen, soft cap", us, kv + 4 * q.numel(), 4.0 * M * H * n * D, like=True)
+        del ks, vs
+        cs = [rnd(M, -(-context // 128) * 128, R) for _ in range(copies(2 * M * context * R))]
+        q = rnd(M, 1, H, R)
+        us = _time_launches([(lambda c=c: ops.latent_attention(q, c, D ** -0.5, context)) for c in cs])
+        yield figure(f"latent attention, decode, {context} rows", us, 2 * M * context * R + 4 * q.numel(), 4.0 * M * H * context * R)
+        del cs
+    ops.attention_check()
+    # ---- matrix memory ----
+    C, E = 2 * MH * (MD + ME), MH * ME
+    state_bytes = 8 * B * MH * MD * ME  # f32, read and written
+    n_cp = 4 if prefill else copies(state_bytes)
+    sts = [ops.MlstmState(B, MH, MD, ME) for _ in range(n_cp)]
+    proj, gates = rnd(B, S, C), torch.randn(B, S, 2 * MH, device="cuda")
+    bias, nw = torch.cat([torch.zeros(MH), 4.0 * torch.ones(MH)]).cuda(), torch.ones(E, device="cuda")
+    past = torch.tensor([context], dtype=torch.int32, device="cuda")
+    us = _time_launches([(lambda st=st: ops.mlstm(proj, gates, bias, nw, st, past, 15.0, 1e-6)) for st in sts])
+    yield figure("matrix memory", us, state_bytes + 2 * M * (C + E), 4.0 * M * MH * MD * ME)
+    del sts
+    # ---- row kernels ----
+    x, sub, w = torch.randn(M, W, device="cuda"), rnd(M, W), torch.ones(W, device="cuda")
+    us = _time_launches([lambda: ops.residual_rms_norm(x, sub, w, 1e-6)] * 16)
+    yield figure("residual + norm", us, M * W * 12, 0.0)
+    pn = (w, torch.zeros(W, device="cuda"))
+    us = _time_launches([lambda: ops.residual_layer_norm(x, sub, pn, 0.5, 1e-5, norm=pn)] * 16)
+    yield figure("post norm + residual + norm", us, M * W * 12, 0.0, like=True)
+    Cq = (H + 2 * G) * D
+    proj, rws = rnd(B, S, Cq), -(-(ck + S) // 128) * 128
+    kc, vc = rnd(B, G, rws, D), rnd(B, G, rws, D)
+    tab, past = torch.rand(max(context, S) + 1, D // 2, device="cuda"), torch.tensor([0 if prefill else context], dtype=torch.int32, device="cuda")
+    us = _time_launches([lambda: ops.rotary_append(proj, past, kc, vc, H, tab, tab)] * 16)
+    yield figure("rotation + head norms + append", us, M * Cq * 4, 0.0)
+    hist, conv, half = rnd(B, 36, Cq), torch.rand(4, Cq, device="cuda"), torch.rand(max(context, S) + 1, D // 4, device="cuda")
+    us = _time_launches([lambda: ops.short_conv_append(proj, past, kc, vc, H, conv, hist, half, half)] * 16)
+    yield figure("convolution + rotation + append", us, M * Cq * 4, 0.0, like=True)
+    lp, cache = rnd(B, S, Q + R), rnd(B, -(-(context + S) // 128) * 128, R)
+    wq, wc = torch.ones(Q, device="cuda"), torch.ones(R, device="cuda")
+    us = _time_launches([lambda: ops.latent_append(lp, past, cache, wq, wc, 1e-6)] * 16)
+    yield figure("latent norms + append", us, M * (Q + R) * 4, 0.0)
+    if int(status.item()):
+        raise RuntimeError(f"dense_matmul: a bounded wait ran out (status {int(status.item())})")
+
+
 def run_case(args):
     def emit(res):
         print(json.dumps(res), flush=True)
@@ -935,6 +1120,15 @@ def run_case(args):
         for name in ([args.block] if args.block else BLOCK_ARCHS):
             for rows in ([args.m] if args.m_given else (1, 32, 2048)):
                 for res in case_block_kernels(name, rows, args.len):
+                    emit(res)
+    elif c == "fimadra":
+        for name in ([args.fimadra] if args.fimadra else FIMADRA_ARCHS):
+            for batch in ([args.b] if args.b_given else (1, 32)):
+                emit(case_fimadra(name, batch, args.len))
+    elif c == "fimadra_kernels":
+        for name in ([args.fimadra] if args.fimadra else FIMADRA_ARCHS):
+            for rows in ([args.m] if args.m_given else (1, 32, 2048)):
+                for res in case_fimadra_kernels(name, rows, args.len):
                     emit(res)
     elif c == "w8a8":
         emit(case_w8a8(args.m, args.n, args.k, args.dtype, args.copies))
@@ -975,6 +1169,7 @@ def main():
     ap.add_argument("--kernel", default="tcgen05_i8", choices=["tcgen05_i8", "mma_sync"])
     ap.add_argument("--layout", default="nk", choices=["nk", "kn"])
     ap.add_argument("--block", choices=sorted(BLOCK_ARCHS), help="one architecture of --case block / block_kernels (default: all)")
+    ap.add_argument("--fimadra", choices=sorted(FIMADRA_ARCHS), help="one architecture of --case fimadra / fimadra_kernels (default: all)")
     ap.add_argument("--arch", default="llama3-8b", choices=["llama3-8b", "tinyllama"])
     ap.add_argument("--option", action="append", default=[], metavar="NAME=VALUE",
                     help="library option set before the run (mynn_b200_set_option), e.g. decode_ring=0, fuse_rope=0, ksplit=4")

@@ -454,6 +454,79 @@ def window_attention(q, k_cache, v_cache, scale, active, window=0, softcap=0.0, 
     return out
 
 
+def chunk_attention(q, k_cache, v_cache, scale, active, window=0, chunk=0, softcap=0.0, head_major=False, plain=False):
+    """window_attention with a chunk mask; head_major: q [Hq, B, Sq, D] and caches [G, B, rows, .].  Returns [B, Sq, Hq, E]."""
+    B, Hq, Sq, D = (q.shape[1], q.shape[0], *q.shape[2:]) if head_major else q.shape
+    G, rows, E = k_cache.shape[0 if head_major else 1], k_cache.shape[2], v_cache.shape[3]
+    out = torch.empty(B, Sq, Hq, E, dtype=q.dtype, device=q.device)
+    ws = attention_workspace(B, Hq, G, D, rows, q.device)
+    ffi.check(ffi.lib().mynn_b200_chunk_attention(_stream(), _ptr(out), _ptr(q), _ptr(k_cache), _ptr(v_cache), scale, softcap, window, chunk, int(head_major),
+                                                  B, Hq, G, Sq, D, E, rows, active, None, _dt(q), _ptr(ws), ws.numel() * ws.element_size(), int(plain)))
+    return out
+
+
+def residual_rms_norm(x, sub, weight, eps, dtype=None):
+    """x += sub, in place (sub may be None); returns x / sqrt(mean(x^2) + eps) * weight in sub's dtype (or ``dtype``), or None without a weight."""
+    dt = dtype or (sub.dtype if sub is not None else x.dtype)
+    out = torch.empty(x.shape, dtype=dt, device=x.device) if weight is not None else None
+    ffi.check(ffi.lib().mynn_b200_residual_rms_norm(_stream(), _ptr(x), _ptr(sub), _ptr(weight), _ptr(out), eps, x.shape[0], x.shape[1],
+                                                    _DT[dt]))
+    return out
+
+
+def rotary_append(proj, past_dev, k_cache, v_cache, heads, cos, sin, halves=True, qk_norm=True, eps=1e-6):
+    """proj [B, S, C] -> q [B, heads, S, D] rotated and normed per head, the new keys (likewise) and values appended to the rings."""
+    B, S, _ = proj.shape
+    G, D, E = k_cache.shape[1], k_cache.shape[3], v_cache.shape[3]
+    q = torch.empty(B, heads, S, D, dtype=proj.dtype, device=proj.device)
+    ffi.check(ffi.lib().mynn_b200_rotary_append(_stream(), _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(proj), _ptr(cos), _ptr(sin), B, S, heads, G, D, E,
+                                                2 * cos.shape[1] if cos is not None else 0, int(halves), int(qk_norm), eps, k_cache.shape[2],
+                                                _ptr(past_dev), _dt(proj)))
+    return q
+
+
+def latent_append(proj, past_dev, cache, q_weight, c_weight, eps):
+    """proj [B, S, Q + R] -> the normed queries' latent [B, S, Q]; the normed other part appended to cache [B, rows, R]."""
+    B, S, C = proj.shape
+    R = cache.shape[2]
+    out = torch.empty(B, S, C - R, dtype=proj.dtype, device=proj.device)
+    ffi.check(ffi.lib().mynn_b200_latent_append(_stream(), _ptr(out), _ptr(cache), _ptr(proj), _ptr(q_weight), _ptr(c_weight), eps, B, S, C - R, R,
+                                                cache.shape[1], _ptr(past_dev), _dt(proj)))
+    return out
+
+
+def latent_attention(q, cache, scale, active, plain=False, workspace=True):
+    """q [B, Sq, H, R] at positions active - Sq .. active - 1 over latents [B, rows, R] that are keys and values; returns [B, Sq, H, R]."""
+    B, Sq, H, R = q.shape
+    out = torch.empty_like(q)
+    n = ffi.lib().mynn_b200_latent_attention_workspace_bytes(B, Sq, H, R, cache.shape[1]) if workspace else 0
+    ws = torch.empty(n, dtype=torch.uint8, device=q.device) if n else None
+    ffi.check(ffi.lib().mynn_b200_latent_attention(_stream(), _ptr(out), _ptr(q), _ptr(cache), scale, B, Sq, H, R, cache.shape[1], active, None, _dt(q),
+                                                   _ptr(ws), n, int(plain)))
+    return out
+
+
+class MlstmState:
+    """Memory, sum vector and running maximum of B sequences (f32 on the device)."""
+
+    def __init__(self, B, H, D, E, device="cuda"):
+        self.mem = torch.zeros(B, H, D, E, device=device)
+        self.sum = torch.zeros(B, H, D, device=device)
+        self.top = torch.zeros(B, H, device=device)
+        self.tickets = torch.zeros(B * H, dtype=torch.int32, device=device)
+
+
+def mlstm(proj, gates, gate_bias, norm_weight, state, past_dev, cap, eps, form=0):
+    """proj [B, S, H (2 D + 2 E)] (q, k, v, output gate), gates f32 [B, S, 2 H] (input, forget); steps ``state``; returns [B, S, H E]."""
+    B, S, _ = proj.shape
+    H, D, E = state.mem.shape[1:]
+    out = torch.empty(B, S, H * E, dtype=proj.dtype, device=proj.device)
+    scratch = torch.empty(B, S, H * E, device=proj.device)
+    ffi.check(ffi.lib().mynn_b200_mlstm(_stream(), _ptr(out), _ptr(state.mem), _ptr(state.sum), _ptr(state.top), _ptr(proj), _ptr(gates), _ptr(gate_bias),
+                                        _ptr(norm_weight), cap, eps, B, S, H, D, E, _ptr(past_dev), _ptr(scratch), _ptr(state.tickets), _dt(proj), form))
+    return out
+
+
 class MoeRouting:
     """Expert choice of M tokens from f32 logits [M, experts] and the products over the chosen experts."""
 
@@ -493,3 +566,26 @@ def dense_matmul(act, w, glu=False, out=None, out_dtype=None, status=None):
     ffi.check(ffi.lib().mynn_b200_dense_matmul(_stream(), _ptr(out), _ptr(act), _ptr(w), act.shape[0], N, act.shape[1], _dt(act), _dt(out), int(glu),
                                                _ptr(status)))
     return out
+
+
+def dense_matmul_heads(act, w, out=None):
+    """act [M, H, K], w [H, N, K] -> [M, H, N]: one product per head."""
+    M, H, K = act.shape
+    N = w.shape[1]
+    if out is None:
+        out = torch.empty(M, H, N, dtype=act.dtype, device=act.device)
+    ffi.check(ffi.lib().mynn_b200_dense_matmul_ex(_stream(), _ptr(out), _ptr(act), _ptr(w), M, N, K, _dt(act), _dt(out), 0, None, 0, 0, 0, H * K, H * N, H,
+                                                  K, N, None))
+    return out
+
+
+def dense_matmul_ex(act, w, act_fn=ffi.ACT_NONE, f32_columns=0, block=0, status=None):
+    """act [M, K] times w [N, K] with act_fn on the sums; the last ``f32_columns`` columns come back as a second tensor in f32; block: the
+    result is [N / block, M, block]."""
+    (M, K), N = act.shape, w.shape[0]
+    main = N - f32_columns
+    out = torch.empty((main // block, M, block) if block else (M, main), dtype=act.dtype, device=act.device)
+    extra = torch.empty(M, f32_columns, device=act.device) if f32_columns else None
+    ffi.check(ffi.lib().mynn_b200_dense_matmul_ex(_stream(), _ptr(out), _ptr(act), _ptr(w), M, N, K, _dt(act), _dt(out), act_fn, _ptr(extra),
+                                                  main if f32_columns else 0, block, M * block, 0, block, 1, 0, 0, _ptr(status)))
+    return (out, extra) if f32_columns else out

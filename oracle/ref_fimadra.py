@@ -1,6 +1,9 @@
 """Plain CPU restatement of the Fimadra decoder: one function per mechanism, float64 (or any numpy dtype), whole sequence
 at once, no cache, no kernels.  Test infrastructure only; it shares nothing with the product path.
 
+``store`` stands for the rounding of activations where a 16-bit implementation stores them (projections, normed rows, what attention and
+memory give, sublayer outputs); left out, nothing is rounded.  Scores, norms, gates, the memory and the residual sum never are.
+
 Notation: T tokens, W model width, per head key size D and value size E, heads H, kv heads G, latent size R.
 """
 from __future__ import annotations
@@ -8,6 +11,16 @@ from __future__ import annotations
 import math
 
 import numpy as np
+
+
+def exact(x):
+    return x
+
+
+def bf16(x):
+    """To the nearest bfloat16 (ties to even), as float64."""
+    u = np.asarray(x, np.float32).view(np.uint32).astype(np.uint64)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) & 0xFFFF0000).astype(np.uint32).view(np.float32).astype(np.float64)
 
 
 def rms(x, eps):
@@ -50,28 +63,25 @@ def softmax_attention(q, k, v, scale, chunk=None):
     return out
 
 
-def attention_mixer(W, p, h, m, eps, positions):
-    H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+def attention_mixer(W, p, h, m, eps, positions, store=exact):
+    H, D, E = m["heads"], m["dim"], m["vdim"]
     T = h.shape[0]
-    q = (h @ W[p + ".mix.q"].T).reshape(T, H, D)
-    k = (h @ W[p + ".mix.k"].T).reshape(T, G, D)
-    v = (h @ W[p + ".mix.v"].T).reshape(T, G, E)
+    q, k, v = (store(h @ W[f"{p}.mix.{n}"].T).reshape(T, -1, d) for n, d in (("q", D), ("k", D), ("v", E)))
     if m.get("rot"):
         f = half_frequencies(m["rot"]["base"], m["rot"]["dims"])
         q, k = rotate_halves(q, positions, f), rotate_halves(k, positions, f)
-    a = softmax_attention(rms(q, eps), rms(k, eps), v, m["scale"], (m.get("mask") or {}).get("size"))
+    a = store(softmax_attention(store(rms(q, eps)), store(rms(k, eps)), v, m["scale"], (m.get("mask") or {}).get("size")))
     return a.reshape(T, H * E) @ W[p + ".mix.o"].T
 
 
-def latent_mixer(W, p, h, m, eps):
+def latent_mixer(W, p, h, m, eps, store=exact):
     H, D, E = m["heads"], m["dim"], m["vdim"]
     T = h.shape[0]
-    cq = rms(h @ W[p + ".mix.dq"].T, eps) * W[p + ".mix.dq.norm"]
-    c = rms(h @ W[p + ".mix.dkv"].T, eps) * W[p + ".mix.dkv.norm"]
-    q = (cq @ W[p + ".mix.uq"].T).reshape(T, H, D)
-    k = (c @ W[p + ".mix.uk"].T).reshape(T, H, D)
-    v = (c @ W[p + ".mix.uv"].T).reshape(T, H, E)
-    return softmax_attention(q, k, v, m["scale"]).reshape(T, H * E) @ W[p + ".mix.o"].T
+    cq, c = (store(rms(store(h @ W[f"{p}.mix.{n}"].T), eps) * W[f"{p}.mix.{n}.norm"]) for n in ("dq", "dkv"))
+    q = store(cq @ W[p + ".mix.uq"].T).reshape(T, H, D)
+    k = store(c @ W[p + ".mix.uk"].T).reshape(T, H, D)
+    v = store(c @ W[p + ".mix.uv"].T).reshape(T, H, E)
+    return store(softmax_attention(q, k, v, m["scale"])).reshape(T, H * E) @ W[p + ".mix.o"].T
 
 
 def log_sigmoid(z):
@@ -101,41 +111,40 @@ def matrix_memory(q, k, v, i_log, f_log, trace=None):
     return out
 
 
-def mlstm_mixer(W, p, h, m, eps):
+def mlstm_mixer(W, p, h, m, eps, store=exact):
     H, D, E, cap = m["heads"], m["dim"], m["vdim"], m["gate_cap"]
     T = h.shape[0]
-    q = (h @ W[p + ".mix.q"].T).reshape(T, H, D) * D ** -0.5
-    k = (h @ W[p + ".mix.k"].T).reshape(T, H, D)
-    v = (h @ W[p + ".mix.v"].T).reshape(T, H, E)
+    q, k, v, z = (store(h @ W[f"{p}.mix.{n}"].T) for n in "qkvg")
+    q, k, v = q.reshape(T, H, D) * D ** -0.5, k.reshape(T, H, D), v.reshape(T, H, E)
     i_log = soft_cap(h @ W[p + ".mix.i"].T + W[p + ".mix.i.b"], cap)
     f_log = log_sigmoid(soft_cap(h @ W[p + ".mix.f"].T + W[p + ".mix.f.b"], cap))
     o = rms(matrix_memory(q, k, v, i_log, f_log), eps).reshape(T, H * E) * W[p + ".mix.norm"]
-    return (o / (1.0 + np.exp(-(h @ W[p + ".mix.g"].T)))) @ W[p + ".mix.o"].T
+    return store(o / (1.0 + np.exp(-z))) @ W[p + ".mix.o"].T
 
 
-def mixer(W, p, h, entry, eps):
+def mixer(W, p, h, entry, eps, store=exact):
     m, kind = entry["mixer"], entry["type"]
     if kind == "attention":
-        return attention_mixer(W, p, h, m, eps, np.arange(h.shape[0]))
+        return attention_mixer(W, p, h, m, eps, np.arange(h.shape[0]), store)
     if kind == "latent_attention":
-        return latent_mixer(W, p, h, m, eps)
+        return latent_mixer(W, p, h, m, eps, store)
     assert kind == "mlstm", kind
-    return mlstm_mixer(W, p, h, m, eps)
+    return mlstm_mixer(W, p, h, m, eps, store)
 
 
 def square_relu(z):
     return np.maximum(z, 0.0) ** 2
 
 
-def forward(cfg, W, tokens, trace=None):
+def forward(cfg, W, tokens, trace=None, store=exact):
     """Logits [T, vocab] of a whole sequence; ``trace`` (a list) receives the residual stream after every layer."""
     eps = cfg["norm"]["eps"]
     x = W["embed"][np.asarray(tokens)].copy()
     for l, entry in enumerate(cfg["layers"]):
         p = f"l{l}"
-        x = x + mixer(W, p, rms(x, eps) * W[p + ".norm1"], entry, eps)
+        x = x + store(mixer(W, p, store(rms(x, eps) * W[p + ".norm1"]), entry, eps, store))
         if entry.get("mlp"):
-            x = x + square_relu((rms(x, eps) * W[p + ".norm2"]) @ W[p + ".mlp.up"].T) @ W[p + ".mlp.down"].T
+            x = x + store(store(square_relu(store(rms(x, eps) * W[p + ".norm2"]) @ W[p + ".mlp.up"].T)) @ W[p + ".mlp.down"].T)
         if trace is not None:
             trace.append(x.copy())
-    return (rms(x, eps) * W["final.norm"]) @ W["head"].T * cfg["logit_scale"]
+    return store(rms(x, eps) * W["final.norm"]) @ W["head"].T * cfg["logit_scale"]
