@@ -510,11 +510,13 @@ int mynn_b200_latent_attention(void *stream, void *out, const void *q, const voi
  *   i = cap(gates_i + bias_i), f = log sigmoid(cap(gates_f + bias_f)), m' = max(f + m, i), a = e^(f + m - m'), w = e^(i - m'),
  *   S' = a S + w k v^T, n' = a n + w k, o = S'^T q~ / (max(|n'.q~|, e^-m') + 1e-6),
  *   out = o / sqrt(mean(o^2) + eps) * norm_weight * sigmoid(z)          (out [B*S, H*E], norm_weight f32 [H*E])
- * State f32 in place: mem [B, H, D, E], sum [B, H, D] (n), top [B, H] (m); taken as zero when *past_dev == 0.  scratch f32 [B*S, H*E];
- * tickets [B*H], zero before the first use.  form 0: by size, 1: token by token, 2: chunkwise on the tensor cores (16-bit). */
+ * State f32 in place: mem [B, H, D, E], sum [B, H, D] (n), top [B, H] (m); taken as zero when *past_dev == 0.  workspace: device scratch of
+ * mynn_b200_mlstm_workspace_bytes, 256-byte aligned; tickets [B*H], zero before the first use.  form 0: by size, 1: token by token, 2: chunkwise
+ * on mma.sync, 3: chunkwise on tcgen05 (both 16-bit); status: device word of the bounded waits (NULL keeps form 3 off). */
+size_t mynn_b200_mlstm_workspace_bytes(int B, int S, int H, int D, int E, int dtype);
 int mynn_b200_mlstm(void *stream, void *out, float *mem, float *sum, float *top, const void *proj, const float *gates, const float *gate_bias,
-                    const float *norm_weight, float cap, float eps, int B, int S, int H, int D, int E, const int32_t *past_dev, float *scratch,
-                    uint32_t *tickets, int dtype, int form);
+                    const float *norm_weight, float cap, float eps, int B, int S, int H, int D, int E, const int32_t *past_dev, void *workspace,
+                    size_t workspace_bytes, uint32_t *tickets, int dtype, int form, int32_t *status);
 /* Expert choice from f32 logits [M, experts]; the workspace (zeroed before its first use) then describes the (token, slot) rows in expert order
  * for mynn_b200_moe_matmul.  weights_out f32 / experts_out int32 [M, top] may be NULL. */
 size_t mynn_b200_moe_workspace_bytes(int M, int experts, int top);

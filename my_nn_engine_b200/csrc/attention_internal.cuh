@@ -49,6 +49,17 @@ __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void *p) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
                  : "r"((uint32_t)__cvta_generic_to_shared(p)));
 }
+// the same from shared-memory addresses
+__device__ __forceinline__ void ldsm4_at(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4t_at(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void copy16_at(uint32_t smem, const void *gmem, bool in) {
+    const int n = in ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem), "l"(gmem), "r"(n) : "memory");
+}
 // 16 bytes global -> shared (cp.async); zeros when !in, without a read
 __device__ __forceinline__ void copy16(void *smem, const void *gmem, bool in) {
     const int n = in ? 16 : 0;
@@ -62,6 +73,14 @@ __device__ __forceinline__ void split_pack(float x, float y, uint32_t &hi, uint3
     const T xl = from_f32<T>(x - to_f32<T>(xh)), yl = from_f32<T>(y - to_f32<T>(yh));
     hi = (uint32_t)reinterpret_cast<const uint16_t &>(xh) | ((uint32_t)reinterpret_cast<const uint16_t &>(yh) << 16);
     lo = (uint32_t)reinterpret_cast<const uint16_t &>(xl) | ((uint32_t)reinterpret_cast<const uint16_t &>(yl) << 16);
+}
+
+template <>
+__device__ __forceinline__ void split_pack<__nv_bfloat16>(float x, float y, uint32_t &hi, uint32_t &lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    hi = reinterpret_cast<const uint32_t &>(h);
+    const __nv_bfloat162 l = __floats2bfloat162_rn(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
+    lo = reinterpret_cast<const uint32_t &>(l);
 }
 
 // cap * tanh(x / cap) = cap - 2 cap / (1 + e^(2 x / cap)); absolute error a few 1e-7 of cap

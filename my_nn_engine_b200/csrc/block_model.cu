@@ -47,7 +47,8 @@ struct BlockModel {
     void *lat_q, *lat_o, *lat_k, *lat_v, *lat_c;  // latent attention: queries and results in latent space, or keys and values; normed queries' latent
     void *lat_ws;
     size_t lat_ws_bytes;
-    float *gates, *mem_o;  // mlstm: gate products, heads before their norm
+    float *gates, *mem_ws;  // mlstm: gate products, workspace
+    size_t mem_ws_bytes;
     unsigned *tickets;
     int32_t *last_rows;  // row of every sequence's last token in a chunk
     // what the rings hold: positions stored since the sequence began, and the most that were ever stored in it
@@ -189,7 +190,8 @@ int block_create(Model &m, void **initializer, void **session_state) {
         }
         if (l.mixer == MYNN_MIX_MLSTM) {
             gn = std::max(gn, R * 2 * (size_t)l.heads);
-            mo = std::max(mo, R * l.heads * (size_t)l.vdim);
+            // not monotonic in the number of tokens: fewer tokens may be cut into more segments
+            for (int s = 1; s <= chunk; s++) mo = std::max(mo, mlstm_workspace_bytes(c.dtype, c.batch, s, l.heads, l.dim, l.vdim));
             tk = std::max(tk, (size_t)c.batch * l.heads);
         }
         if (l.dense_ff) pairs_ff = std::max(pairs_ff, R * (size_t)l.dense_ff);
@@ -213,7 +215,7 @@ int block_create(Model &m, void **initializer, void **session_state) {
                  o_gat = area(gat * esz), o_route = area(route), o_z = area(zn * 4), o_log = area((size_t)m.head_capacity * c.vocab * 4),
                  o_rows = area((size_t)m.head_capacity * 4), o_last = area((size_t)c.batch * 4), o_pairs = area((size_t)c.batch * 8 * 16), o_aws = area(aws),
                  o_stat = area(512), o_lq = area(lq * esz), o_lo = area(lq * esz), o_lk = area(lk * esz), o_lv = area(lv * esz), o_lc = area(lc_n * esz),
-                 o_lws = area(lws), o_gates = area(gn * 4), o_mo = area(mo * 4), o_tk = area(tk * 4);
+                 o_lws = area(lws), o_gates = area(gn * 4), o_mo = area(mo), o_tk = area(tk * 4);
     cudaError_t e = cudaMalloc(&m.arena, off);
     if (e != cudaSuccess) return fail(MYNN_E_CUDA, "model_init: cudaMalloc(%zu) failed: %s", off, cudaGetErrorString(e));
     MYNN_CUDA_OK(cudaMemset(m.arena, 0, off));
@@ -247,7 +249,8 @@ int block_create(Model &m, void **initializer, void **session_state) {
     b.lat_ws = a + o_lws;
     b.lat_ws_bytes = lws;
     b.gates = (float *)(a + o_gates);
-    b.mem_o = (float *)(a + o_mo);
+    b.mem_ws = (float *)(a + o_mo);
+    b.mem_ws_bytes = mo;
     b.tickets = (unsigned *)(a + o_tk);
     return MYNN_OK;
 }
@@ -419,11 +422,13 @@ static int mix_mlstm(Model &m, cudaStream_t st, const BlockLayer &L, const Block
     p.cap = l.gate_cap;
     p.eps = b.c.norm_eps;
     p.mem = (float *)run.kc, p.sum = (float *)run.vc, p.top = (float *)run.hist;
-    p.o = b.mem_o;
+    p.workspace = b.mem_ws;
+    p.workspace_bytes = b.mem_ws_bytes;
     p.ticket = b.tickets;
     p.out = b.attn;
     p.B = b.c.batch, p.S = S, p.H = l.heads, p.D = l.dim, p.E = l.vdim;
     p.past = m.past_dev;
+    p.status = (int *)m.gemm_ws;
     return launch_mlstm(st, dt, p);
 }
 

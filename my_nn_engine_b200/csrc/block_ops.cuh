@@ -160,15 +160,18 @@ struct MlstmStep {
     const float *gates = nullptr, *gate_bias = nullptr, *norm_w = nullptr;
     float cap = 1.f, eps = 0.f;
     float *mem = nullptr, *sum = nullptr, *top = nullptr;
-    float *o = nullptr;          // scratch f32 [B * S, H E]
+    float *workspace = nullptr;  // mlstm_workspace_bytes; begins with o, f32 [B * S, H E]
+    size_t workspace_bytes = 0;
     unsigned *ticket = nullptr;  // scratch [B * H], zero between calls
     void *out = nullptr;         // [B * S, H E]
     int B = 0, S = 0, H = 0, D = 0, E = 0;
     const int32_t *past = nullptr;
-    int form = 0;                // 0: by size, 1: token by token, 2: chunkwise (16-bit)
+    int form = 0;                // 0: by size, 1: token by token, 2: chunkwise on mma.sync, 3: chunkwise on tcgen05 (both 16-bit)
+    int *status = nullptr;       // status word of the bounded waits (tcgen05 form only)
 };
 int launch_mlstm(cudaStream_t st, int dtype, const MlstmStep &p);
 bool mlstm_chunkwise_supported(int dtype, const MlstmStep &p);
+size_t mlstm_workspace_bytes(int dtype, int B, int S, int H, int D, int E);
 
 // ---- moe_route.cu ----------------------------------------------------------------------------------------------------
 // Expert choice of M tokens from f32 logits [M, E]: s = softmax(z); of `groups` equal groups of neighbouring experts the `keep`

@@ -3,9 +3,11 @@
 //
 // latent_append_kernel      norms the two latents of a new token (queries', and the one that is cached) and appends the second.
 // latent_attention_kernel   16-bit, R = 128, 256 or 512: few queries per sequence (decode, short portions).  A CTA takes 16 or 32 heads of
-//                           one query and a range of positions, in tiles of 64 that cp.async keeps two of in shared memory.  The
-//                           tile is the B operand of both products: scores (warps deal out heads and keys) and weighted sum (warps
-//                           deal out the R columns).  Weights enter the second product as a high part and its remainder.
+//                           one query and a range of positions, in tiles of 32 that cp.async keeps two of in shared memory (two CTAs share an SM, one computes while the other waits).  The
+//                           tile is the B operand of both products.  For the scores a warp takes 16 heads and a part of the R columns, so
+//                           that its queries stay in registers; the parts meet in shared memory.  For the weighted sum the warps deal
+//                           out the R columns; weights are rounded to 16 bits there, as in the prefill kernels (mma.sync sets the
+//                           pace with 32 heads: a second product for the remainders costs 20 % of the kernel).
 // latent_merge_kernel       combines the ranges of a query.
 // Everything else (32-bit, other R) goes to the window attention kernel for any sizes, keys and values being the same rows.
 #include <algorithm>
@@ -55,7 +57,7 @@ int launch_latent_append(cudaStream_t st, int dtype, const LatentAppend &p) {
 }
 
 // ---- attention -------------------------------------------------------------------------------------------------------
-constexpr int kLatKeys = 64, kLatThreads = 256, kLatMaxSplits = 64;
+constexpr int kLatKeys = 32, kLatThreads = 256, kLatMaxSplits = 64;
 
 struct LatParams {
     void *out;
@@ -68,21 +70,27 @@ struct LatParams {
 
 template <typename T, int R, int MT>
 struct LatSmem {
-    static constexpr int LD = R + 8, LP = kLatKeys + 8;
+    static constexpr int LD = R + 8, LP = kLatKeys + 8, LS = kLatKeys + 4, PARTS = 8 / MT;
     T c[2][kLatKeys][LD];
-    T q[16 * MT][LD];
-    T p_hi[16 * MT][LP], p_lo[16 * MT][LP];
-    float s[16 * MT][kLatKeys + 4];
+    T p[16 * MT][LP];
+    float s[PARTS][16 * MT][LS];  // partial scores
     float alpha[16 * MT], m[16 * MT], l[16 * MT];
 };
 
+__device__ __forceinline__ float lat_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 // grid (splits, B * Sq, head groups)
 template <typename T, int R, int MT>
-__global__ void __launch_bounds__(kLatThreads, 1) latent_attention_kernel(const LatParams p) {
+__global__ void __launch_bounds__(kLatThreads, 2) latent_attention_kernel(const LatParams p) {
     extern __shared__ __align__(16) uint8_t lat_smem[];
     using Sm = LatSmem<T, R, MT>;
     Sm &sm = *reinterpret_cast<Sm *>(lat_smem);
     constexpr int HB = 16 * MT, PIECES = R / 8, NT = R / 64;  // heads of the CTA, 16-byte pieces of a row, column tiles per warp
+    constexpr int PARTS = Sm::PARTS, RP = R / PARTS, KS = RP / 16;  // the scores' contraction is cut into parts
     pdl_trigger();
     pdl_wait();
     const int split = blockIdx.x, query = blockIdx.y, b = query / p.Sq, s_i = query - b * p.Sq, h0 = blockIdx.z * HB;
@@ -95,21 +103,34 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attention_kernel(const 
     const int heads = min(HB, p.H - h0);
     const size_t slot0 = (size_t)query * p.H + h0;
 
+    // a thread copies one 16-byte column of every RC-th row
+    constexpr int RC = kLatThreads / PIECES;
+    const int c_row = threadIdx.x / PIECES, c_col = (threadIdx.x % PIECES) * 8;
+    const uint32_t c_dst = (uint32_t)__cvta_generic_to_shared(&sm.c[0][c_row][c_col]);
     auto fetch = [&](int j) {
-        for (int i = threadIdx.x; i < kLatKeys * PIECES; i += kLatThreads) {
-            const int r = i / PIECES, d = (i % PIECES) * 8, pos = beg + j * kLatKeys + r;
-            const bool in = pos < end;
-            copy16(&sm.c[j & 1][r][d], cache + (size_t)(in ? pos : 0) * R + d, in);
+        const T *src = cache + (size_t)(beg + j * kLatKeys + c_row) * R + c_col;
+        const uint32_t dst = c_dst + (j & 1) * (uint32_t)sizeof(sm.c[0]);
+        const int left = end - beg - j * kLatKeys - c_row;
+#pragma unroll
+        for (int i = 0; i < kLatKeys / RC; i++) {
+            const bool in = i * RC < left;
+            copy16_at(dst + i * RC * Sm::LD * (uint32_t)sizeof(T), in ? src + (size_t)i * RC * R : cache, in);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     if (tiles > 0) fetch(0);
+    const int mt = warp % MT, part = warp / MT;
+    uint32_t qa[KS][4];  // queries of 16 heads, RP columns
     {
-        const T *q = reinterpret_cast<const T *>(p.q) + slot0 * R;
-        for (int i = threadIdx.x; i < HB * PIECES; i += kLatThreads) {
-            const int r = i / PIECES, d = (i % PIECES) * 8;
-            *reinterpret_cast<uint4 *>(&sm.q[r][d]) = r < heads ? *reinterpret_cast<const uint4 *>(q + (size_t)r * R + d) : make_uint4(0u, 0u, 0u, 0u);
-        }
+        const int r0 = 16 * mt + gq;
+        const T *q = reinterpret_cast<const T *>(p.q) + slot0 * R + part * RP + 2 * t4;
+#pragma unroll
+        for (int ks = 0; ks < KS; ks++)
+#pragma unroll
+            for (int x = 0; x < 4; x++) {
+                const int r = r0 + 8 * (x & 1);
+                qa[ks][x] = r < heads ? *reinterpret_cast<const uint32_t *>(q + (size_t)r * R + 16 * ks + 8 * (x >> 1)) : 0u;
+            }
         if (threadIdx.x < HB) sm.m[threadIdx.x] = -INFINITY, sm.l[threadIdx.x] = 0.f;
     }
     float o[MT][NT][4];
@@ -117,69 +138,79 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attention_kernel(const 
     for (int i = 0; i < MT; i++)
 #pragma unroll
         for (int j = 0; j < NT; j++) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
+    const int c0 = warp * (R / 8);
+    const uint32_t k_addr = (uint32_t)__cvta_generic_to_shared(&sm.c[0][(lane & 7) + 8 * (lane >> 4)][part * RP + 8 * ((lane >> 3) & 1)]);
+    const uint32_t v_addr = (uint32_t)__cvta_generic_to_shared(&sm.c[0][lane & 15][c0 + 8 * (lane >> 4)]);
+    const uint32_t p_addr = (uint32_t)__cvta_generic_to_shared(&sm.p[lane & 15][8 * (lane >> 4)]);
+    constexpr uint32_t kRow = Sm::LD * sizeof(T), kPRow = Sm::LP * sizeof(T);
 
     for (int j = 0; j < tiles; j++) {
-        const int buf = j & 1, key0 = beg + j * kLatKeys;
+        const int key0 = beg + j * kLatKeys;
+        const uint32_t buf = (j & 1) * (uint32_t)sizeof(sm.c[0]);
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();  // tile j is there, tile j - 1 has been read by all
         if (j + 1 < tiles) fetch(j + 1);
-        // ---- scores ----
-        if constexpr (MT == 2) {  // 16 heads x 16 keys per warp
-            const int mt = warp & 1, k0 = (warp >> 1) * 16;
-            float sc[2][2][4] = {};
-#pragma unroll 4
-            for (int kk = 0; kk < R; kk += 32) {
+        // ---- scores: 16 heads x 64 keys over RP columns ----
+        {
+            float sc[kLatKeys / 8][4];
 #pragma unroll
-                for (int u = 0; u < 2; u++) {  // two chains
-                    uint32_t qa[4], kb[4];
-                    ldsm4(qa, &sm.q[16 * mt + (lane & 15)][kk + 16 * u + 8 * (lane >> 4)]);
-                    ldsm4(kb, &sm.c[buf][k0 + (lane & 7) + 8 * (lane >> 4)][kk + 16 * u + 8 * ((lane >> 3) & 1)]);
-                    mma_kv<T>(sc[u][0], qa[0], qa[1], qa[2], qa[3], kb[0], kb[1]);
-                    mma_kv<T>(sc[u][1], qa[0], qa[1], qa[2], qa[3], kb[2], kb[3]);
+            for (int n = 0; n < kLatKeys / 8; n++) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+#pragma unroll
+            for (int ks = 0; ks < KS; ks++)
+#pragma unroll
+                for (int n = 0; n < kLatKeys / 16; n++) {
+                    uint32_t kb[4];  // 16 keys: (first 8, k low), (first 8, k high), (last 8, ..)
+                    ldsm4_at(kb, k_addr + buf + n * 16 * kRow + ks * 32);
+                    mma_kv<T>(sc[2 * n], qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3], kb[0], kb[1]);
+                    mma_kv<T>(sc[2 * n + 1], qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3], kb[2], kb[3]);
                 }
+#pragma unroll
+            for (int n = 0; n < kLatKeys / 8; n++) {
+                *reinterpret_cast<float2 *>(&sm.s[part][16 * mt + gq][8 * n + 2 * t4]) = make_float2(sc[n][0], sc[n][1]);
+                *reinterpret_cast<float2 *>(&sm.s[part][16 * mt + gq + 8][8 * n + 2 * t4]) = make_float2(sc[n][2], sc[n][3]);
             }
-#pragma unroll
-            for (int n = 0; n < 2; n++)
-#pragma unroll
-                for (int x = 0; x < 4; x++) sm.s[16 * mt + gq + 8 * (x >> 1)][k0 + 8 * n + 2 * t4 + (x & 1)] = sc[0][n][x] + sc[1][n][x];
-        } else {  // 16 heads x 8 keys per warp
-            const int k0 = warp * 8;
-            float sc[2][4] = {};
-#pragma unroll 4
-            for (int kk = 0; kk < R; kk += 32) {
-                uint32_t qa[4], qb[4], kb[4];
-                ldsm4(qa, &sm.q[lane & 15][kk + 8 * (lane >> 4)]);
-                ldsm4(qb, &sm.q[lane & 15][kk + 16 + 8 * (lane >> 4)]);
-                ldsm4(kb, &sm.c[buf][k0 + (lane & 7)][kk + 8 * (lane >> 3)]);
-                mma_kv<T>(sc[0], qa[0], qa[1], qa[2], qa[3], kb[0], kb[1]);
-                mma_kv<T>(sc[1], qb[0], qb[1], qb[2], qb[3], kb[2], kb[3]);
-            }
-#pragma unroll
-            for (int x = 0; x < 4; x++) sm.s[gq + 8 * (x >> 1)][k0 + 2 * t4 + (x & 1)] = sc[0][x] + sc[1][x];
         }
         __syncthreads();
-        // ---- softmax: a warp takes 2 MT heads, two keys per lane ----
+        // ---- softmax: a warp takes 2 MT heads, one key per lane ----
+        {
+            float w[2 * MT], top[2 * MT], sum[2 * MT], al[2 * MT];
 #pragma unroll
-        for (int i = 0; i < 2 * MT; i++) {
-            const int r = warp * 2 * MT + i, k = 2 * lane;
-            const float2 raw = *reinterpret_cast<const float2 *>(&sm.s[r][k]);
-            const float x0 = key0 + k < end ? raw.x * p.scale_log2 : -INFINITY, x1 = key0 + k + 1 < end ? raw.y * p.scale_log2 : -INFINITY;
-            const float m_old = sm.m[r], m_new = fmaxf(m_old, warp_max(fmaxf(x0, x1)));  // finite: the tile has a key
-            const float w0 = exp2f(x0 - m_new), w1 = exp2f(x1 - m_new), al = exp2f(m_old - m_new), sum = warp_sum(w0 + w1);
-            uint32_t hi, lo;
-            split_pack<T>(w0, w1, hi, lo);
-            *reinterpret_cast<uint32_t *>(&sm.p_hi[r][k]) = hi;
-            *reinterpret_cast<uint32_t *>(&sm.p_lo[r][k]) = lo;
-            __syncwarp();
+            for (int i = 0; i < 2 * MT; i++) {
+                const int r = warp * 2 * MT + i;
+                float x = 0.f;
+#pragma unroll
+                for (int q = 0; q < PARTS; q++) x += sm.s[q][r][lane];
+                top[i] = w[i] = key0 + lane < end ? x * p.scale_log2 : -INFINITY;
+            }
+#pragma unroll
+            for (int s = 16; s > 0; s >>= 1)
+#pragma unroll
+                for (int i = 0; i < 2 * MT; i++) top[i] = fmaxf(top[i], __shfl_xor_sync(0xffffffffu, top[i], s));
+#pragma unroll
+            for (int i = 0; i < 2 * MT; i++) {
+                const int r = warp * 2 * MT + i;
+                const float m_old = sm.m[r], m_new = fmaxf(m_old, top[i]);  // finite: the tile has a key
+                w[i] = lat_exp2(w[i] - m_new), al[i] = lat_exp2(m_old - m_new);
+                top[i] = m_new;
+                sum[i] = w[i];
+                sm.p[r][lane] = from_f32<T>(w[i]);
+            }
+#pragma unroll
+            for (int s = 16; s > 0; s >>= 1)
+#pragma unroll
+                for (int i = 0; i < 2 * MT; i++) sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], s);
             if (lane == 0) {
-                sm.m[r] = m_new;
-                sm.l[r] = sm.l[r] * al + sum;
-                sm.alpha[r] = al;
+#pragma unroll
+                for (int i = 0; i < 2 * MT; i++) {
+                    const int r = warp * 2 * MT + i;
+                    sm.m[r] = top[i];
+                    sm.l[r] = sm.l[r] * al[i] + sum[i];
+                    sm.alpha[r] = al[i];
+                }
             }
         }
         __syncthreads();
         // ---- weighted sum: R / 8 columns per warp ----
-        const int c0 = warp * (R / 8);
 #pragma unroll
         for (int i = 0; i < MT; i++) {
             const float a0 = sm.alpha[16 * i + gq], a1 = sm.alpha[16 * i + gq + 8];
@@ -190,16 +221,13 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attention_kernel(const 
         for (int kk = 0; kk < kLatKeys; kk += 16) {
             uint32_t vb[NT / 2][4];
 #pragma unroll
-            for (int n = 0; n < NT / 2; n++) ldsm4t(vb[n], &sm.c[buf][kk + (lane & 15)][c0 + 16 * n + 8 * (lane >> 4)]);
+            for (int n = 0; n < NT / 2; n++) ldsm4t_at(vb[n], v_addr + buf + kk * kRow + n * 32);
 #pragma unroll
             for (int i = 0; i < MT; i++) {
-                uint32_t ph[4], pl[4];
-                ldsm4(ph, &sm.p_hi[16 * i + (lane & 15)][kk + 8 * (lane >> 4)]);
-                ldsm4(pl, &sm.p_lo[16 * i + (lane & 15)][kk + 8 * (lane >> 4)]);
+                uint32_t ph[4];
+                ldsm4_at(ph, p_addr + 16 * i * kPRow + kk * 2);
 #pragma unroll
                 for (int n = 0; n < NT; n++) mma_kv<T>(o[i][n], ph[0], ph[1], ph[2], ph[3], vb[n >> 1][2 * (n & 1)], vb[n >> 1][2 * (n & 1) + 1]);
-#pragma unroll
-                for (int n = 0; n < NT; n++) mma_kv<T>(o[i][n], pl[0], pl[1], pl[2], pl[3], vb[n >> 1][2 * (n & 1)], vb[n >> 1][2 * (n & 1) + 1]);
             }
         }
     }
@@ -232,45 +260,68 @@ __global__ void __launch_bounds__(kLatThreads, 1) latent_attention_kernel(const 
     }
 }
 
-// one CTA per (query, head), two neighbouring columns per thread (R / 2 threads)
+// one CTA per (query, head), two neighbouring columns per thread (R / 2 threads); eight splits in flight
 template <typename T>
 __global__ void __launch_bounds__(256) latent_merge_kernel(const LatParams p, int R) {
+    __shared__ float f[kLatMaxSplits];
+    __shared__ float total;
     pdl_trigger();
     pdl_wait();
     const size_t slot = blockIdx.x;
     const float *ml = p.ws_ml + slot * p.splits * 2, *o = p.ws_o + slot * p.splits * R + 2 * threadIdx.x;
-    float mx = -INFINITY;
-    for (int s = 0; s < p.splits; s++) mx = fmaxf(mx, ml[2 * s]);
-    float L = 0.f;
-    float2 acc = make_float2(0.f, 0.f);
-#pragma unroll 4
-    for (int s = 0; s < p.splits; s++) {
-        if (ml[2 * s] == -INFINITY) continue;
-        const float f = exp2f(ml[2 * s] - mx);
-        const float2 v = *reinterpret_cast<const float2 *>(o + (size_t)s * R);
-        L += f * ml[2 * s + 1];
-        acc.x += f * v.x, acc.y += f * v.y;
+    float2 v[8];
+    auto load = [&](int s0) {
+#pragma unroll
+        for (int j = 0; j < 8; j++) v[j] = s0 + j < p.splits ? *reinterpret_cast<const float2 *>(o + (size_t)(s0 + j) * R) : make_float2(0.f, 0.f);
+    };
+    load(0);  // travels while the factors are formed; a split without positions left stale numbers, which meet a factor of 0
+    if (threadIdx.x < 32) {
+        float m[kLatMaxSplits / 32], mx = -INFINITY, L = 0.f;
+#pragma unroll
+        for (int j = 0; j < kLatMaxSplits / 32; j++) {
+            const int s = threadIdx.x + 32 * j;
+            m[j] = s < p.splits ? ml[2 * s] : -INFINITY;
+            mx = fmaxf(mx, m[j]);
+        }
+        mx = warp_max(mx);
+#pragma unroll
+        for (int j = 0; j < kLatMaxSplits / 32; j++) {
+            const int s = threadIdx.x + 32 * j;
+            const float w = m[j] == -INFINITY ? 0.f : lat_exp2(m[j] - mx);
+            if (s < p.splits) L += w * ml[2 * s + 1];
+            f[s] = w;
+        }
+        L = warp_sum(L);
+        if (threadIdx.x == 0) total = L;
     }
-    const float inv = L > 0.f ? 1.0f / L : 0.f;
+    __syncthreads();
+    float2 acc = make_float2(0.f, 0.f);
+    for (int s0 = 0; s0 < p.splits; s0 += 8) {
+        if (s0) load(s0);
+#pragma unroll
+        for (int j = 0; j < 8; j++)
+            if (s0 + j < p.splits && f[s0 + j] != 0.f) acc.x += f[s0 + j] * v[j].x, acc.y += f[s0 + j] * v[j].y;
+    }
+    const float inv = total > 0.f ? 1.0f / total : 0.f;
     T two[2] = {from_f32<T>(acc.x * inv), from_f32<T>(acc.y * inv)};
     *reinterpret_cast<uint32_t *>(reinterpret_cast<T *>(p.out) + slot * R + 2 * threadIdx.x) = *reinterpret_cast<const uint32_t *>(two);
 }
 
 static int lat_splits(int queries, int groups, int rows_bound) {
-    int s = 148 / (queries * groups);
-    s = std::min(s, rows_bound / (2 * kLatKeys));  // at least two tiles each
+    int s = 296 / (queries * groups);
+    s = std::min(s, rows_bound / (4 * kLatKeys));  // at least four tiles each
     return std::max(1, std::min(s, kLatMaxSplits));
 }
 // 16 heads per CTA while that still leaves SMs idle, else 32 (the latents are then read half as often)
 static int lat_head_tiles(int queries, int H, int rows_bound) {
     if (H <= 16) return 1;
     const int g = (H + 31) / 32;
-    return queries * g * lat_splits(queries, g, rows_bound) < 74 ? 1 : 2;
+    return queries * g * lat_splits(queries, g, rows_bound) < 148 ? 1 : 2;
 }
 
 size_t latent_attention_workspace_bytes(int B, int Sq, int H, int R, int cache_rows) {
     const long long queries = (long long)B * Sq;
-    if (queries <= 0 || queries > 148) return 0;
+    if (queries <= 0 || queries > 296) return 0;
     const int s = std::max(lat_splits((int)queries, (H + 15) / 16, cache_rows), lat_splits((int)queries, (H + 31) / 32, cache_rows));
     return s == 1 ? 0 : (size_t)queries * H * s * (R + 2) * sizeof(float) + 256;
 }

@@ -117,7 +117,8 @@ SIGNATURES = {
     "mynn_b200_latent_append": (c_int, [c_void_p] * 6 + [c_float] + [c_int] * 5 + [c_void_p, c_int]),
     "mynn_b200_latent_attention_workspace_bytes": (c_size_t, [c_int] * 5),
     "mynn_b200_latent_attention": (c_int, [c_void_p] * 4 + [c_float] + [c_int] * 6 + [c_void_p, c_int, c_void_p, c_size_t, c_int]),
-    "mynn_b200_mlstm": (c_int, [c_void_p] * 9 + [c_float, c_float] + [c_int] * 5 + [c_void_p] * 3 + [c_int, c_int]),
+    "mynn_b200_mlstm_workspace_bytes": (c_size_t, [c_int] * 6),
+    "mynn_b200_mlstm": (c_int, [c_void_p] * 9 + [c_float, c_float] + [c_int] * 5 + [c_void_p, c_void_p, c_size_t, c_void_p] + [c_int, c_int, c_void_p]),
     "mynn_b200_dense_matmul_ex": (c_int, [c_void_p] * 4 + [c_int] * 6 + [c_void_p, c_int, c_int, ctypes.c_longlong, c_int, c_int, c_int, ctypes.c_longlong, ctypes.c_longlong, c_void_p]),
     "mynn_b200_moe_workspace_bytes": (c_size_t, [c_int, c_int, c_int]),
     "mynn_b200_moe_route": (c_int, [c_void_p, c_void_p, c_size_t, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int]),

@@ -514,6 +514,7 @@ class MlstmState:
         self.sum = torch.zeros(B, H, D, device=device)
         self.top = torch.zeros(B, H, device=device)
         self.tickets = torch.zeros(B * H, dtype=torch.int32, device=device)
+        self.status = torch.zeros(1, dtype=torch.int32, device=device)
 
 
 def mlstm(proj, gates, gate_bias, norm_weight, state, past_dev, cap, eps, form=0):
@@ -521,9 +522,10 @@ def mlstm(proj, gates, gate_bias, norm_weight, state, past_dev, cap, eps, form=0
     B, S, _ = proj.shape
     H, D, E = state.mem.shape[1:]
     out = torch.empty(B, S, H * E, dtype=proj.dtype, device=proj.device)
-    scratch = torch.empty(B, S, H * E, device=proj.device)
+    n = ffi.lib().mynn_b200_mlstm_workspace_bytes(B, S, H, D, E, _dt(proj))
+    ws = torch.empty(n, dtype=torch.uint8, device=proj.device)
     ffi.check(ffi.lib().mynn_b200_mlstm(_stream(), _ptr(out), _ptr(state.mem), _ptr(state.sum), _ptr(state.top), _ptr(proj), _ptr(gates), _ptr(gate_bias),
-                                        _ptr(norm_weight), cap, eps, B, S, H, D, E, _ptr(past_dev), _ptr(scratch), _ptr(state.tickets), _dt(proj), form))
+                                        _ptr(norm_weight), cap, eps, B, S, H, D, E, _ptr(past_dev), _ptr(ws), n, _ptr(state.tickets), _dt(proj), form, _ptr(state.status)))
     return out
 
 

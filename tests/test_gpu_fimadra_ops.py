@@ -201,8 +201,9 @@ def memory_oracle(proj, gates, bias, norm, H, D, E, cap, eps):
     return np.array(outs), states
 
 
-MEMORY_SHAPES = [("f32", 3, 20, 28, [0, 1]), ("f32", 1, 70, 33, [1]), ("bf16", 2, 48, 40, [1, 2]), ("bf16", 1, 64, 96, [0, 1, 2]), ("bf16", 2, 128, 72, [1, 2]),
-                 ("bf16", 1, 200, 32, [1, 2]), ("bf16", 1, 256, 64, [2]), ("f16", 1, 32, 32, [1, 2]), ("f32", 1, 300, 16, [1]), ("bf16", 2, 6, 10, [0, 1])]
+MEMORY_SHAPES = [("f32", 3, 20, 28, [0, 1]), ("f32", 1, 70, 33, [1]), ("bf16", 2, 48, 40, [1, 2]), ("bf16", 1, 64, 96, [0, 1, 2]), ("bf16", 2, 128, 72, [1, 2, 3]),
+                 ("bf16", 1, 200, 32, [1, 2]), ("bf16", 1, 200, 136, [0, 2]), ("bf16", 1, 256, 136, [0, 2, 3]), ("f16", 1, 32, 32, [1, 2]), ("f16", 1, 128, 264, [2, 3]),
+                 ("f32", 1, 300, 16, [1]), ("bf16", 2, 6, 10, [0, 1])]
 
 
 @pytest.mark.parametrize("dt,H,D,E,forms", MEMORY_SHAPES)
@@ -223,27 +224,28 @@ def test_matrix_memory_in_portions(dt, H, D, E, forms):
             for b in range(B):
                 for name, mine, ref in zip(("S", "n", "m"), (st.mem, st.sum, st.top), states[b]):
                     # 32-bit whatever the dtype; chunkwise products keep the values as two 16-bit parts
-                    close(host(mine)[b], ref, 4e-6 if form != 2 else 2e-5 if dt == "bf16" else 4e-6, f"state {name}, form {form}, {sizes}")
-            assert not st.tickets.any()
+                    close(host(mine)[b], ref, 4e-6 if dt == "f32" or form == 1 else 2e-5, f"state {name}, form {form}, {sizes}")
+            assert not st.tickets.any() and not st.status.any()
 
 
-@pytest.mark.parametrize("form", [1, 2])
+@pytest.mark.parametrize("form", [1, 2, 3])
 @pytest.mark.parametrize("forget,spread", [(-30.0, 3.0), (30.0, 0.1), (0.0, 40.0)], ids=["forgets all", "keeps all", "gates at their caps"])
 def test_matrix_memory_with_extreme_gates(form, forget, spread):
     rng = np.random.default_rng(4)
-    H, D, E, cap = 2, 32, 48, 15.0
-    proj, gates, bias, norm = memory_inputs(rng, 1, 150, H, D, E, "bf16", forget, spread)
+    H, D, E, cap = 2, 128, 72, 15.0
+    proj, gates, bias, norm = memory_inputs(rng, 1, 350, H, D, E, "bf16", forget, spread)
     want, _ = memory_oracle(proj, gates, bias, norm, H, D, E, cap, 1e-6)
     st = ops.MlstmState(1, H, D, E)
-    got = [ops.mlstm(proj[:, a:b].contiguous(), gates[:, a:b].contiguous(), bias, norm, st, past(a), cap, 1e-6, form) for a, b in ((0, 100), (100, 150))]
+    got = [ops.mlstm(proj[:, a:b].contiguous(), gates[:, a:b].contiguous(), bias, norm, st, past(a), cap, 1e-6, form) for a, b in ((0, 300), (300, 350))]
     close(host(torch.cat(got, 1)), want, TOL["bf16"])
+    assert not st.status.any()
 
 
 def test_matrix_memory_remembers_one_token_over_hundreds():
     """A key that comes once, far back, and a query for it at the end: the state in between has to carry it."""
     rng = np.random.default_rng(5)
-    H, D, E, T = 1, 64, 32, 700
-    for dt, forms in (("f32", [1]), ("bf16", [1, 2])):
+    H, D, E, T = 1, 128, 64, 700
+    for dt, forms in (("f32", [1]), ("bf16", [1, 2, 3])):
         x = 0.05 * rng.standard_normal((1, T, 2 * H * (D + E)))
         u = np.sign(rng.standard_normal(D))
         x[0, 3, D:2 * D] = u
@@ -257,6 +259,24 @@ def test_matrix_memory_remembers_one_token_over_hundreds():
             st = ops.MlstmState(1, H, D, E)
             got = [ops.mlstm(proj[:, a:b].contiguous(), gates[:, a:b].contiguous(), bias, norm, st, past(a), 10.0, 1e-6, form) for a, b in ((0, 640), (640, 699), (699, 700))]
             close(host(got[-1])[0, -1], want[0, -1], TOL[dt])
+
+
+def test_matrix_memory_in_segments_equals_token_by_token():
+    """Long prompts over few heads are cut into segments that run side by side; two prompts in a row, state and outputs."""
+    rng = np.random.default_rng(6)
+    for H, D, E, S in ((1, 256, 128, 1100), (3, 128, 200, 700), (2, 64, 64, 900)):
+        proj, gates, bias, norm = memory_inputs(rng, 1, S, H, D, E, "bf16", 5.0, 1.0)
+        ref, refs = ops.MlstmState(1, H, D, E), []
+        for a, b in ((0, S - 130), (S - 130, S)):
+            refs.append(ops.mlstm(proj[:, a:b].contiguous(), gates[:, a:b].contiguous(), bias, norm, ref, past(a), 12.0, 1e-6, 1))
+        for form in (0, 2):
+            st = ops.MlstmState(1, H, D, E)
+            for (a, b), want in zip(((0, S - 130), (S - 130, S)), refs):
+                got = ops.mlstm(proj[:, a:b].contiguous(), gates[:, a:b].contiguous(), bias, norm, st, past(a), 12.0, 1e-6, form)
+                close(host(got), host(want), 1e-2, f"{H} {D} {E} form {form} from {a}")
+            for mine, theirs in ((st.mem, ref.mem), (st.sum, ref.sum), (st.top, ref.top)):
+                close(host(mine), host(theirs), 3e-5)
+            assert not st.status.any()
 
 
 # ---- products ----
