@@ -226,7 +226,7 @@ __global__ void __launch_bounds__(kStreamWarps * 32, MT * RT * (GLU ? 2 : 1) <= 
 template <typename T, typename O>
 static int run_stream(cudaStream_t st, const GemmView &v, int rows, int groups, int glu) {
     const int mt = rows <= 8 ? 1 : rows <= 16 ? 2 : 4;
-    const bool wide = !glu && (mt > 1 || v.N >= 16 * 148 * 4) && v.N >= 32 * 100;
+    const bool wide = !glu && (v.batch > 1 ? v.N * (long long)v.batch >= 32 * 148 * 2 : (mt > 1 || v.N >= 16 * 148 * 4) && v.N >= 32 * 100);
     const dim3 grid((v.N + (wide ? 31 : 15)) / (wide ? 32 : 16), groups);
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;

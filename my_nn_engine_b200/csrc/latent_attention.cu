@@ -18,10 +18,11 @@
 
 namespace mynn {
 
-// grid (2, B * S): the queries' latent, the cached latent
-template <typename T>
-__global__ void __launch_bounds__(128) latent_append_kernel(const LatentAppend p) {
-    __shared__ float red[4];
+// grid (2, B * S): the queries' latent, the cached latent.  V: elements a thread moves at a time (8 needs 16-bit rows of 16-byte pieces); up
+// to 2 V elements per thread stay in registers between the sum and the store, longer rows are read again.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) latent_append_kernel(const LatentAppend p) {
+    __shared__ float red[8];
     pdl_trigger();
     pdl_wait();
     const int row = blockIdx.y, second = blockIdx.x, W = second ? p.R : p.Q;
@@ -34,16 +35,59 @@ __global__ void __launch_bounds__(128) latent_append_kernel(const LatentAppend p
     } else {
         out = reinterpret_cast<T *>(p.q_out) + (size_t)row * p.Q;
     }
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < W; i += 128) {
-        const float v = to_f32<T>(x[i]);
-        ss += v * v;
+    auto load = [&](int i, float (&v)[V]) {
+        if constexpr (V == 8) {
+            const uint4 r = *reinterpret_cast<const uint4 *>(x + i);
+            const T *e = reinterpret_cast<const T *>(&r);
+#pragma unroll
+            for (int k = 0; k < 8; k++) v[k] = to_f32<T>(e[k]);
+        } else {
+            v[0] = to_f32<T>(x[i]);
+        }
+    };
+    float v[2][V], ss = 0.f;
+    const int step = 256 * V, i0 = threadIdx.x * V;
+#pragma unroll
+    for (int j = 0; j < 2; j++)
+        if (i0 + j * step < W) {
+            load(i0 + j * step, v[j]);
+#pragma unroll
+            for (int k = 0; k < V; k++) ss += v[j][k] * v[j][k];
+        }
+    for (int i = i0 + 2 * step; i < W; i += step) {
+        float u[V];
+        load(i, u);
+#pragma unroll
+        for (int k = 0; k < V; k++) ss += u[k] * u[k];
     }
     ss = warp_sum(ss);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
     __syncthreads();
-    const float inv = 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / (float)W + p.eps);
-    for (int i = threadIdx.x; i < W; i += 128) out[i] = from_f32<T>(to_f32<T>(x[i]) * inv * w[i]);
+    float total = 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; k++) total += red[k];
+    const float inv = 1.0f / sqrtf(total / (float)W + p.eps);
+    auto store = [&](int i, const float (&u)[V]) {
+        if constexpr (V == 8) {
+            const float4 a = *reinterpret_cast<const float4 *>(w + i), b = *reinterpret_cast<const float4 *>(w + i + 4);
+            const float g[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+            uint4 r;
+            T *e = reinterpret_cast<T *>(&r);
+#pragma unroll
+            for (int k = 0; k < 8; k++) e[k] = from_f32<T>(u[k] * inv * g[k]);
+            *reinterpret_cast<uint4 *>(out + i) = r;
+        } else {
+            out[i] = from_f32<T>(u[0] * inv * w[i]);
+        }
+    };
+#pragma unroll
+    for (int j = 0; j < 2; j++)
+        if (i0 + j * step < W) store(i0 + j * step, v[j]);
+    for (int i = i0 + 2 * step; i < W; i += step) {
+        float u[V];
+        load(i, u);
+        store(i, u);
+    }
 }
 
 int launch_latent_append(cudaStream_t st, int dtype, const LatentAppend &p) {
@@ -51,7 +95,14 @@ int launch_latent_append(cudaStream_t st, int dtype, const LatentAppend &p) {
     if (!dtype_ok(dtype)) return fail(MYNN_E_ARG, "latent_append: bad dtype %d", dtype);
     if (!p.proj || !p.wq || !p.wc || !p.q_out || !p.cache || !p.past) return fail(MYNN_E_ARG, "latent_append: null pointer");
     if ((long long)p.B * p.S > 65535) return fail(MYNN_E_UNSUPPORTED, "latent_append: %d x %d tokens in one step", p.B, p.S);
-    MYNN_DISPATCH_DTYPE(dtype, T, { latent_append_kernel<T><<<dim3(2, p.B * p.S), 128, 0, st>>>(p); });
+    const dim3 grid(2, p.B * p.S);
+    const uintptr_t a = (uintptr_t)p.proj | (uintptr_t)p.q_out | (uintptr_t)p.cache | (uintptr_t)p.wq | (uintptr_t)p.wc;
+    if (dtype != MYNN_F32 && p.Q % 8 == 0 && p.R % 8 == 0 && a % 16 == 0) {
+        if (dtype == MYNN_BF16) latent_append_kernel<__nv_bfloat16, 8><<<grid, 256, 0, st>>>(p);
+        else latent_append_kernel<__half, 8><<<grid, 256, 0, st>>>(p);
+    } else {
+        MYNN_DISPATCH_DTYPE(dtype, T, { latent_append_kernel<T, 1><<<grid, 256, 0, st>>>(p); });
+    }
     MYNN_LAUNCH_OK("latent_append_kernel");
     return MYNN_OK;
 }
@@ -344,7 +395,7 @@ static int run_latent(cudaStream_t st, const LatParams &l, int queries) {
     kern<<<dim3(l.splits, queries, l.groups), kLatThreads, smem, st>>>(l);
     MYNN_LAUNCH_OK("latent_attention_kernel");
     if (l.splits > 1) {
-        latent_merge_kernel<T><<<(unsigned)((long long)queries * l.H), R / 2, 0, st>>>(l, R);
+        MYNN_CUDA_OK(launch_dependent(latent_merge_kernel<T>, dim3((unsigned)((long long)queries * l.H)), dim3(R / 2), 0, st, l, R));
         MYNN_LAUNCH_OK("latent_merge_kernel");
     }
     return MYNN_OK;

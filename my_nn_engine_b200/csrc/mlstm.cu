@@ -85,9 +85,10 @@ __global__ void __launch_bounds__(256) mlstm_out_kernel(const MlstmStep p) {
     gated_row<T>(p, row, h, 1.0f / sqrtf(warp_sum(ss) / (float)p.E + p.eps), lane, 32);
 }
 
-// grid (ceil(E / 32), H, B), 256 threads.  Warp w holds rows [w NR, (w + 1) NR) of the memory tile, lane l column l.
-template <typename T, int NR>
-__global__ void __launch_bounds__(kScanWarps * 32, NR <= 16 ? 4 : NR <= 32 ? 3 : 1) mlstm_scan_kernel(const MlstmStep p) {
+// grid (ceil(E / 32), H, B), 256 threads.  Warp w holds rows [w NR, (w + 1) NR) of the memory tile, lane l column l.  ONE: a single token, which
+// is all about reading and writing the memory: four CTAs per SM keep enough of it on its way.
+template <typename T, int NR, bool ONE>
+__global__ void __launch_bounds__(kScanWarps * 32, ONE && NR <= 32 ? 4 : 1) mlstm_scan_kernel(const MlstmStep p) {
     constexpr int DP = kScanWarps * NR;  // rows with padding
     __shared__ __align__(16) float sm_q[2][DP], sm_k[2][DP];
     __shared__ float sm_num[2][kScanWarps][kScanCols], sm_den[2][kScanWarps];
@@ -129,7 +130,7 @@ __global__ void __launch_bounds__(kScanWarps * 32, NR <= 16 ? 4 : NR <= 32 ? 3 :
     };
     stage(0);
     __syncthreads();
-    for (int t = 0; t < p.S; t++) {
+    for (int t = 0; t < p.S; t++) {  // also with ONE a loop: all of the memory's reads are then on their way in front of it
         const size_t row = (size_t)b * p.S + t;
         const float v = in ? to_f32<T>(reinterpret_cast<const T *>(p.proj)[row * C + (size_t)2 * p.H * p.D + (size_t)h * p.E + col]) : 0.f;
         const float gi = capped(p.gates[row * 2 * p.H + h] + bias_i, p.cap), gf = log_sigmoid(capped(p.gates[row * 2 * p.H + p.H + h] + bias_f, p.cap));
@@ -157,7 +158,7 @@ __global__ void __launch_bounds__(kScanWarps * 32, NR <= 16 ? 4 : NR <= 32 ? 3 :
         den = warp_sum(den);
         sm_num[t & 1][warp][lane] = num;
         if (lane == 0) sm_den[t & 1][warp] = den;
-        if (t + 1 < p.S) stage(t + 1);
+        if (!ONE && t + 1 < p.S) stage(t + 1);
         __syncthreads();
         if (warp == 0 && in) {
             float a = 0.f, d = 0.f;
@@ -178,7 +179,7 @@ __global__ void __launch_bounds__(kScanWarps * 32, NR <= 16 ? 4 : NR <= 32 ? 3 :
         if (r < NR && d < p.D) p.sum[(size_t)pair * p.D + d] = n[j];
     }
     if (threadIdx.x == 0) p.top[pair] = m;
-    if (p.S == 1) {
+    if constexpr (ONE) {
         const float *o = p.workspace + (size_t)pair * p.E;
         float ss = 0.f;
         for (int e = threadIdx.x; e < p.E; e += blockDim.x) {
@@ -559,15 +560,15 @@ static int run_out(cudaStream_t st, const MlstmStep &p) {
     return MYNN_OK;
 }
 
-template <typename T>
+template <typename T, bool ONE>
 static int run_scan(cudaStream_t st, const MlstmStep &p) {
     const dim3 grid((p.E + kScanCols - 1) / kScanCols, p.H, p.B);
-    if (p.D <= 64) mlstm_scan_kernel<T, 8><<<grid, 256, 0, st>>>(p);
-    else if (p.D <= 128) mlstm_scan_kernel<T, 16><<<grid, 256, 0, st>>>(p);
-    else if (p.D <= 256) mlstm_scan_kernel<T, 32><<<grid, 256, 0, st>>>(p);
-    else mlstm_scan_kernel<T, 64><<<grid, 256, 0, st>>>(p);
+    if (p.D <= 64) mlstm_scan_kernel<T, 8, ONE><<<grid, 256, 0, st>>>(p);
+    else if (p.D <= 128) mlstm_scan_kernel<T, 16, ONE><<<grid, 256, 0, st>>>(p);
+    else if (p.D <= 256) mlstm_scan_kernel<T, 32, ONE><<<grid, 256, 0, st>>>(p);
+    else mlstm_scan_kernel<T, 64, ONE><<<grid, 256, 0, st>>>(p);
     MYNN_LAUNCH_OK("mlstm_scan_kernel");
-    return p.S == 1 ? MYNN_OK : run_out<T>(st, p);
+    return ONE ? MYNN_OK : run_out<T>(st, p);
 }
 
 template <typename T, int KD, bool OUT>
@@ -619,8 +620,8 @@ int launch_mlstm(cudaStream_t st, int dtype, const MlstmStep &p) {
     if (p.workspace_bytes < (size_t)p.B * p.S * p.H * p.E * sizeof(float)) return fail(MYNN_E_ARG, "mlstm: workspace of %zu bytes", p.workspace_bytes);
     const bool can = mlstm_chunkwise_supported(dtype, p);
     if ((p.form == 2 && !can) || (p.form == 3 && !(can && mlstm_tc_supported(dtype, p)))) return fail(MYNN_E_UNSUPPORTED, "mlstm: not a shape of the chunkwise kernel");
-    if (p.form >= 2 || (p.form == 0 && can && p.S > 16)) return dtype == MYNN_BF16 ? run_chunk_any<__nv_bfloat16>(st, dtype, p) : run_chunk_any<__half>(st, dtype, p);
-    MYNN_DISPATCH_DTYPE(dtype, T, { return run_scan<T>(st, p); });
+    if (p.form >= 2 || (p.form == 0 && can && p.S > 12)) return dtype == MYNN_BF16 ? run_chunk_any<__nv_bfloat16>(st, dtype, p) : run_chunk_any<__half>(st, dtype, p);
+    MYNN_DISPATCH_DTYPE(dtype, T, { return p.S == 1 ? run_scan<T, true>(st, p) : run_scan<T, false>(st, p); });
     return MYNN_OK;
 }
 
