@@ -3,7 +3,7 @@
 //
 // latent_append_kernel      norms the two latents of a new token (queries', and the one that is cached) and appends the second.
 // latent_attention_kernel   16-bit, R = 128, 256 or 512: few queries per sequence (decode, short portions).  A CTA takes 16 or 32 heads of
-//                           one query and a range of positions, in tiles of 32 that cp.async keeps two of in shared memory (two CTAs share an SM, one computes while the other waits).  The
+//                           one query and a range of positions, in tiles of 64 that cp.async keeps two of in shared memory.  The
 //                           tile is the B operand of both products.  For the scores a warp takes 16 heads and a part of the R columns, so
 //                           that its queries stay in registers; the parts meet in shared memory.  For the weighted sum the warps deal
 //                           out the R columns; weights are rounded to 16 bits there, as in the prefill kernels (mma.sync sets the
@@ -108,7 +108,8 @@ int launch_latent_append(cudaStream_t st, int dtype, const LatentAppend &p) {
 }
 
 // ---- attention -------------------------------------------------------------------------------------------------------
-constexpr int kLatKeys = 32, kLatThreads = 256, kLatMaxSplits = 64;
+constexpr int kLatKeys = 64, kLatMaxSplits = 64;
+constexpr int lat_warps(int R) { return R == 128 ? 8 : 16; }  // a warp takes at least 16 columns of the weighted sum
 
 struct LatParams {
     void *out;
@@ -121,7 +122,7 @@ struct LatParams {
 
 template <typename T, int R, int MT>
 struct LatSmem {
-    static constexpr int LD = R + 8, LP = kLatKeys + 8, LS = kLatKeys + 4, PARTS = 8 / MT;
+    static constexpr int LD = R + 8, LP = kLatKeys + 8, LS = kLatKeys + 8, WARPS = lat_warps(R), PARTS = WARPS / MT;
     T c[2][kLatKeys][LD];
     T p[16 * MT][LP];
     float s[PARTS][16 * MT][LS];  // partial scores
@@ -136,11 +137,11 @@ __device__ __forceinline__ float lat_exp2(float x) {
 
 // grid (splits, B * Sq, head groups)
 template <typename T, int R, int MT>
-__global__ void __launch_bounds__(kLatThreads, 2) latent_attention_kernel(const LatParams p) {
+__global__ void __launch_bounds__(lat_warps(R) * 32, R == 128 ? 2 : 1) latent_attention_kernel(const LatParams p) {
     extern __shared__ __align__(16) uint8_t lat_smem[];
     using Sm = LatSmem<T, R, MT>;
     Sm &sm = *reinterpret_cast<Sm *>(lat_smem);
-    constexpr int HB = 16 * MT, PIECES = R / 8, NT = R / 64;  // heads of the CTA, 16-byte pieces of a row, column tiles per warp
+    constexpr int WARPS = Sm::WARPS, HB = 16 * MT, PIECES = R / 8, NT = R / (8 * WARPS);  // heads of the CTA, 16-byte pieces of a row, column tiles per warp
     constexpr int PARTS = Sm::PARTS, RP = R / PARTS, KS = RP / 16;  // the scores' contraction is cut into parts
     pdl_trigger();
     pdl_wait();
@@ -155,7 +156,7 @@ __global__ void __launch_bounds__(kLatThreads, 2) latent_attention_kernel(const 
     const size_t slot0 = (size_t)query * p.H + h0;
 
     // a thread copies one 16-byte column of every RC-th row
-    constexpr int RC = kLatThreads / PIECES;
+    constexpr int RC = WARPS * 32 / PIECES;
     const int c_row = threadIdx.x / PIECES, c_col = (threadIdx.x % PIECES) * 8;
     const uint32_t c_dst = (uint32_t)__cvta_generic_to_shared(&sm.c[0][c_row][c_col]);
     auto fetch = [&](int j) {
@@ -189,7 +190,7 @@ __global__ void __launch_bounds__(kLatThreads, 2) latent_attention_kernel(const 
     for (int i = 0; i < MT; i++)
 #pragma unroll
         for (int j = 0; j < NT; j++) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
-    const int c0 = warp * (R / 8);
+    const int c0 = warp * (R / WARPS);
     const uint32_t k_addr = (uint32_t)__cvta_generic_to_shared(&sm.c[0][(lane & 7) + 8 * (lane >> 4)][part * RP + 8 * ((lane >> 3) & 1)]);
     const uint32_t v_addr = (uint32_t)__cvta_generic_to_shared(&sm.c[0][lane & 15][c0 + 8 * (lane >> 4)]);
     const uint32_t p_addr = (uint32_t)__cvta_generic_to_shared(&sm.p[lane & 15][8 * (lane >> 4)]);
@@ -222,38 +223,45 @@ __global__ void __launch_bounds__(kLatThreads, 2) latent_attention_kernel(const 
             }
         }
         __syncthreads();
-        // ---- softmax: a warp takes 2 MT heads, one key per lane ----
+        // ---- softmax: a warp takes RW heads, two keys per lane ----
         {
-            float w[2 * MT], top[2 * MT], sum[2 * MT], al[2 * MT];
+            constexpr int RW = HB / WARPS;
+            float w0[RW], w1[RW], top[RW], sum[RW], al[RW];
+            const int k = 2 * lane;
 #pragma unroll
-            for (int i = 0; i < 2 * MT; i++) {
-                const int r = warp * 2 * MT + i;
-                float x = 0.f;
+            for (int i = 0; i < RW; i++) {
+                const int r = warp * RW + i;
+                float x0 = 0.f, x1 = 0.f;
 #pragma unroll
-                for (int q = 0; q < PARTS; q++) x += sm.s[q][r][lane];
-                top[i] = w[i] = key0 + lane < end ? x * p.scale_log2 : -INFINITY;
+                for (int q = 0; q < PARTS; q++) {
+                    const float2 v = *reinterpret_cast<const float2 *>(&sm.s[q][r][k]);
+                    x0 += v.x, x1 += v.y;
+                }
+                w0[i] = key0 + k < end ? x0 * p.scale_log2 : -INFINITY, w1[i] = key0 + k + 1 < end ? x1 * p.scale_log2 : -INFINITY;
+                top[i] = fmaxf(w0[i], w1[i]);
             }
 #pragma unroll
             for (int s = 16; s > 0; s >>= 1)
 #pragma unroll
-                for (int i = 0; i < 2 * MT; i++) top[i] = fmaxf(top[i], __shfl_xor_sync(0xffffffffu, top[i], s));
+                for (int i = 0; i < RW; i++) top[i] = fmaxf(top[i], __shfl_xor_sync(0xffffffffu, top[i], s));
 #pragma unroll
-            for (int i = 0; i < 2 * MT; i++) {
-                const int r = warp * 2 * MT + i;
+            for (int i = 0; i < RW; i++) {
+                const int r = warp * RW + i;
                 const float m_old = sm.m[r], m_new = fmaxf(m_old, top[i]);  // finite: the tile has a key
-                w[i] = lat_exp2(w[i] - m_new), al[i] = lat_exp2(m_old - m_new);
+                w0[i] = lat_exp2(w0[i] - m_new), w1[i] = lat_exp2(w1[i] - m_new), al[i] = lat_exp2(m_old - m_new);
                 top[i] = m_new;
-                sum[i] = w[i];
-                sm.p[r][lane] = from_f32<T>(w[i]);
+                sum[i] = w0[i] + w1[i];
+                T two[2] = {from_f32<T>(w0[i]), from_f32<T>(w1[i])};
+                *reinterpret_cast<uint32_t *>(&sm.p[r][k]) = *reinterpret_cast<const uint32_t *>(two);
             }
 #pragma unroll
             for (int s = 16; s > 0; s >>= 1)
 #pragma unroll
-                for (int i = 0; i < 2 * MT; i++) sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], s);
+                for (int i = 0; i < RW; i++) sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], s);
             if (lane == 0) {
 #pragma unroll
-                for (int i = 0; i < 2 * MT; i++) {
-                    const int r = warp * 2 * MT + i;
+                for (int i = 0; i < RW; i++) {
+                    const int r = warp * RW + i;
                     sm.m[r] = top[i];
                     sm.l[r] = sm.l[r] * al[i] + sum[i];
                     sm.alpha[r] = al[i];
@@ -261,7 +269,7 @@ __global__ void __launch_bounds__(kLatThreads, 2) latent_attention_kernel(const 
             }
         }
         __syncthreads();
-        // ---- weighted sum: R / 8 columns per warp ----
+        // ---- weighted sum: R / WARPS columns per warp ----
 #pragma unroll
         for (int i = 0; i < MT; i++) {
             const float a0 = sm.alpha[16 * i + gq], a1 = sm.alpha[16 * i + gq + 8];
@@ -292,14 +300,14 @@ __global__ void __launch_bounds__(kLatThreads, 2) latent_attention_kernel(const 
             const float l = sm.l[r];
             if (p.splits == 1) {
                 const float inv = l > 0.f ? 1.0f / l : 0.f;
-                T *out = reinterpret_cast<T *>(p.out) + (slot0 + r) * R + warp * (R / 8) + 2 * t4;
+                T *out = reinterpret_cast<T *>(p.out) + (slot0 + r) * R + warp * (R / WARPS) + 2 * t4;
 #pragma unroll
                 for (int n = 0; n < NT; n++) {
                     T two[2] = {from_f32<T>(o[i][n][2 * x] * inv), from_f32<T>(o[i][n][2 * x + 1] * inv)};
                     *reinterpret_cast<uint32_t *>(out + 8 * n) = *reinterpret_cast<const uint32_t *>(two);
                 }
             } else if (tiles > 0) {
-                float *out = p.ws_o + ((slot0 + r) * p.splits + split) * R + warp * (R / 8) + 2 * t4;
+                float *out = p.ws_o + ((slot0 + r) * p.splits + split) * R + warp * (R / WARPS) + 2 * t4;
 #pragma unroll
                 for (int n = 0; n < NT; n++) *reinterpret_cast<float2 *>(out + 8 * n) = make_float2(o[i][n][2 * x], o[i][n][2 * x + 1]);
             }
@@ -359,20 +367,20 @@ __global__ void __launch_bounds__(256) latent_merge_kernel(const LatParams p, in
 }
 
 static int lat_splits(int queries, int groups, int rows_bound) {
-    int s = 296 / (queries * groups);
-    s = std::min(s, rows_bound / (4 * kLatKeys));  // at least four tiles each
+    int s = 148 / (queries * groups);
+    s = std::min(s, rows_bound / (2 * kLatKeys));  // at least four tiles each
     return std::max(1, std::min(s, kLatMaxSplits));
 }
 // 16 heads per CTA while that still leaves SMs idle, else 32 (the latents are then read half as often)
 static int lat_head_tiles(int queries, int H, int rows_bound) {
     if (H <= 16) return 1;
     const int g = (H + 31) / 32;
-    return queries * g * lat_splits(queries, g, rows_bound) < 148 ? 1 : 2;
+    return queries * g * lat_splits(queries, g, rows_bound) < 74 ? 1 : 2;
 }
 
 size_t latent_attention_workspace_bytes(int B, int Sq, int H, int R, int cache_rows) {
     const long long queries = (long long)B * Sq;
-    if (queries <= 0 || queries > 296) return 0;
+    if (queries <= 0 || queries > 148) return 0;
     const int s = std::max(lat_splits((int)queries, (H + 15) / 16, cache_rows), lat_splits((int)queries, (H + 31) / 32, cache_rows));
     return s == 1 ? 0 : (size_t)queries * H * s * (R + 2) * sizeof(float) + 256;
 }
@@ -392,7 +400,7 @@ static int run_latent(cudaStream_t st, const LatParams &l, int queries) {
         MYNN_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         attr_set = true;
     }
-    kern<<<dim3(l.splits, queries, l.groups), kLatThreads, smem, st>>>(l);
+    kern<<<dim3(l.splits, queries, l.groups), lat_warps(R) * 32, smem, st>>>(l);
     MYNN_LAUNCH_OK("latent_attention_kernel");
     if (l.splits > 1) {
         MYNN_CUDA_OK(launch_dependent(latent_merge_kernel<T>, dim3((unsigned)((long long)queries * l.H)), dim3(R / 2), 0, st, l, R));
