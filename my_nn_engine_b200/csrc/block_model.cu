@@ -344,7 +344,6 @@ static int mix_latent(Model &m, cudaStream_t st, const BlockLayer &L, const Bloc
     BlockModel &b = *m.blocks;
     const mynn_b200_block &l = L.c;
     const int B = b.c.batch, M = B * S, H = b.c.hidden, dt = b.c.dtype, R = l.kv_rank;
-    const size_t esz = dtype_size(dt);
     RC(launch_dense_gemm(st, dt, plain_product(m, b.proj, dt, b.h, L.qkv, M, columns(l), H)));
     LatentAppend la;
     la.proj = b.proj;
@@ -384,15 +383,14 @@ static int mix_latent(Model &m, cudaStream_t st, const BlockLayer &L, const Bloc
     q.out_block = l.dim, q.out_block_stride = (long long)M * l.dim, q.ldo = l.dim;
     RC(launch_dense_gemm(st, dt, q));
     const long long rows = (long long)B * l.cache_rows;
-    for (int i = 0; i < B; i++) {
-        const void *c = (const char *)run.kc + (size_t)i * l.cache_rows * R * esz;
-        DenseGemm k = plain_product(m, (char *)b.lat_k + (size_t)i * l.cache_rows * l.dim * esz, dt, c, L.uk, b.stored, l.heads * l.dim, R);
-        k.out_block = l.dim, k.out_block_stride = rows * l.dim, k.ldo = l.dim;
-        RC(launch_dense_gemm(st, dt, k));
-        DenseGemm v = plain_product(m, (char *)b.lat_v + (size_t)i * l.cache_rows * l.vdim * esz, dt, c, L.uv, b.stored, l.heads * l.vdim, R);
-        v.out_block = l.vdim, v.out_block_stride = rows * l.vdim, v.ldo = l.vdim;
-        RC(launch_dense_gemm(st, dt, v));
-    }
+    DenseGemm k = plain_product(m, b.lat_k, dt, run.kc, L.uk, b.stored, l.heads * l.dim, R);
+    k.out_block = l.dim, k.out_block_stride = rows * l.dim, k.ldo = l.dim;
+    k.row_groups = B, k.group_rows = l.cache_rows;
+    RC(launch_dense_gemm(st, dt, k));
+    DenseGemm v = plain_product(m, b.lat_v, dt, run.kc, L.uv, b.stored, l.heads * l.vdim, R);
+    v.out_block = l.vdim, v.out_block_stride = rows * l.vdim, v.ldo = l.vdim;
+    v.row_groups = B, v.group_rows = l.cache_rows;
+    RC(launch_dense_gemm(st, dt, v));
     WindowAttention at;
     at.out = b.attn;
     at.q = b.q;

@@ -204,6 +204,8 @@ int launch_moe_route(cudaStream_t st, const MoeRoute &r, const float *logits, in
 //   out_block: column n of row m is stored at (n / out_block) * out_block_stride + m * ldo + n % out_block (one block per head, say)
 //   batch:    independent products side by side (rows of act lda apart, product z at act + z * act_stride, w + z * N * K,
 //             out + z * out_stride); not on the tensor-memory kernel
+//   row_groups: the rows come in that many groups of M, group r at rows r * group_rows .. of act and out (the live rows of every sequence's
+//             cache, say)
 enum { kActNone = MYNN_ACT_NONE, kActSquareRelu = MYNN_ACT_SQUARE_RELU };
 struct DenseGemm {
     void *out = nullptr;
@@ -223,6 +225,8 @@ struct DenseGemm {
     int lda = 0, ldo = 0;       // row strides in elements, 0: K and N (n_main with out_f32)
     int batch = 1;
     long long act_stride = 0, out_stride = 0;
+    int row_groups = 1;
+    long long group_rows = 0;
 };
 __device__ __forceinline__ float dense_act(float v, int fn) {
     if (fn == kActSquareRelu) {

@@ -263,6 +263,19 @@ int launch_dense_gemm(cudaStream_t st, int dtype, const DenseGemm &g) {
     if (!dtype_ok(dtype) || (g.out_dtype != dtype && g.out_dtype != MYNN_F32)) return fail(MYNN_E_ARG, "dense_matmul: bad dtypes %d -> %d", dtype, g.out_dtype);
     if (g.M == 0) return MYNN_OK;
     if (!g.out || !g.act || !g.w) return fail(MYNN_E_ARG, "dense_matmul: null pointer");
+    if (g.row_groups > 1) {
+        if (g.route || g.batch > 1 || g.out_f32 || g.group_rows < g.M) return fail(MYNN_E_ARG, "dense_matmul: %d groups of %d rows, %lld apart", g.row_groups, g.M, g.group_rows);
+        if (!dense_gemm_tc_supported(dtype, g)) {  // one after the other
+            for (int r = 0; r < g.row_groups; r++) {
+                DenseGemm one = g;
+                one.row_groups = 1;
+                one.act = (const char *)g.act + (size_t)r * g.group_rows * (g.lda ? g.lda : g.K) * dtype_size(dtype);
+                one.out = (char *)g.out + (size_t)r * g.group_rows * (g.ldo ? g.ldo : g.N) * dtype_size(g.out_dtype);
+                if (int rc = launch_dense_gemm(st, dtype, one)) return rc;
+            }
+            return MYNN_OK;
+        }
+    }
     if (g.out_f32 ? g.n_main <= 0 || g.n_main > g.N : g.n_main != 0) return fail(MYNN_E_ARG, "dense_matmul: %d of %d columns in the main output", g.n_main, g.N);
     if (g.batch < 1 || g.batch > 65535 || (g.batch > 1 && (g.route || g.out_f32)) || (g.route && (g.out_f32 || g.out_block || g.lda || g.ldo)) ||
         (g.glu && (g.act_fn || g.out_f32)) || g.out_block < 0)

@@ -37,6 +37,8 @@ struct DgParams {
     int ldo, n_main, act_fn, out_block;           // see DenseGemm; out_block 0: none
     long long out_block_stride;
     float *out_f32;
+    int groups, group_tiles;                      // dense: groups of rows and row tiles of each; 0: one group
+    long long group_rows;                         // distance of the groups' first rows
     int *status;
 };
 
@@ -92,12 +94,14 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
     tc_fence_after();
     const uint32_t tmem_base = tmem_slot;
     pdl_wait();  // activations and the tile list come from the preceding kernels
-    const int m_tiles = p.m_tiles_dev ? *p.m_tiles_dev : (p.M + kDgRows - 1) / kDgRows;
+    const int m_tiles = p.m_tiles_dev ? *p.m_tiles_dev : p.group_tiles ? p.group_tiles * p.groups : (p.M + kDgRows - 1) / kDgRows;
     const int total = m_tiles * p.n_tiles;
     auto give_up = [&](int code) {
         atomicExch(&abort_flag, 1);
         atomicExch(p.status, code);
     };
+    auto group_base = [&](int mt) { return p.group_tiles ? (int)((mt / p.group_tiles) * p.group_rows) : 0; };
+    auto dense_row = [&](int mt) { return group_base(mt) + (p.group_tiles ? mt % p.group_tiles : mt) * kDgRows; };
     auto locate = [&](int tile, int &mt, int &nt) {
         if (p.row_fastest) nt = tile / m_tiles, mt = tile - nt * m_tiles;
         else mt = tile / p.n_tiles, nt = tile - mt * p.n_tiles;
@@ -113,7 +117,7 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
             for (int tile = blockIdx.x; tile < total && ok; tile += gridDim.x) {
                 int mt, nt;
                 locate(tile, mt, nt);
-                const int e = p.tile_e ? p.tile_e[mt] : 0, row = p.tile_row ? p.tile_row[mt] : mt * kDgRows;
+                const int e = p.tile_e ? p.tile_e[mt] : 0, row = p.tile_row ? p.tile_row[mt] : dense_row(mt);
                 const int wrow = e * (GLU ? 2 * p.N : p.N) + nt * NT;
                 for (int kb = 0; kb < kblocks; kb++, kc++) {
                     const int s = kc % kDgStages, use = kc / kDgStages;
@@ -184,8 +188,8 @@ dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
             const int buf = it & 1, use = it >> 1;
             int mt, nt;
             locate(tile, mt, nt);
-            const int r0 = p.tile_row ? p.tile_row[mt] : mt * kDgRows;
-            const int end = p.tile_e ? p.off[p.tile_e[mt] + 1] : p.M;
+            const int r0 = p.tile_row ? p.tile_row[mt] : dense_row(mt);
+            const int end = p.tile_e ? p.off[p.tile_e[mt] + 1] : group_base(mt) + p.M;
             int ok = 1;
             if (lane == 0) {
                 ok = mbar_wait_spin(&acc_full[buf], use & 1, &abort_flag) ? 1 : 0;
@@ -254,7 +258,7 @@ __global__ void __launch_bounds__(256) gather_places_kernel(uint4 *out, const ui
 bool dense_gemm_tc_supported(int dtype, const DenseGemm &g) {
     if (dtype == MYNN_F32 || !g.status || !tensor_map_api_available() || g.K % 8 || g.batch > 1 || (g.lda && g.lda != g.K) || (((uintptr_t)g.act | (uintptr_t)g.w) % 16)) return false;
     const long long wrows = (long long)g.experts * g.N * (g.glu ? 2 : 1), arows = g.route ? (long long)g.M * g.top : g.M;
-    if (wrows >= (1ll << 31) || arows >= (1ll << 31)) return false;
+    if (wrows >= (1ll << 31) || arows >= (1ll << 31) || g.row_groups * g.group_rows >= (1ll << 31)) return false;
     if (!g.route) return g.M > 32;
     if (g.gather && (!g.gather_ws || (uintptr_t)g.gather_ws % 16)) return false;
     return arows >= 16ll * g.experts && g.M > 32;  // enough rows per expert for a 128-row tile to beat passes over its weights
@@ -289,7 +293,8 @@ int launch_dense_gemm_tc(cudaStream_t st, int dtype, const DenseGemm &g) {
     }
     CUtensorMap ma, mw;
     const uint64_t row_bytes = (uint64_t)g.K * 2;
-    if (int rc = make_map(&ma, act, (uint64_t)arows, row_bytes, row_bytes, kDgRows)) return rc;
+    const uint64_t map_rows = g.row_groups > 1 ? (uint64_t)((g.row_groups - 1) * g.group_rows + g.M) : (uint64_t)arows;
+    if (int rc = make_map(&ma, act, map_rows, row_bytes, row_bytes, kDgRows)) return rc;
     if (int rc = make_map(&mw, g.w, (uint64_t)wrows, row_bytes, row_bytes, g.glu ? kDgCols / 2 : kDgCols)) return rc;
     DgParams p = {};
     p.out = g.out;
@@ -304,6 +309,12 @@ int launch_dense_gemm_tc(cudaStream_t st, int dtype, const DenseGemm &g) {
     p.out_block_stride = g.out_block_stride;
     p.out_f32 = g.out_f32;
     long long m_bound = (g.M + kDgRows - 1) / kDgRows;
+    if (g.row_groups > 1) {
+        p.groups = g.row_groups;
+        p.group_tiles = (int)m_bound;
+        p.group_rows = g.group_rows;
+        m_bound *= g.row_groups;
+    }
     if (g.route) {
         p.off = g.route->off;
         p.tile_e = g.route->tile_e;

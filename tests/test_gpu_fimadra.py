@@ -151,16 +151,18 @@ def test_a_recurrent_state_does_not_go_back():
 
 @pytest.mark.parametrize("dtype", ["f32", "bf16"])
 @pytest.mark.parametrize("name", sorted(fm.ALL))
-def test_batch_against_each_alone(name, dtype):
+@pytest.mark.parametrize("sizes", [[64, 37, 2] + [1] * 47, [20, 109, 150, 1, 20]], ids=["decoding", "portions"])
+def test_batch_against_each_alone(name, dtype, sizes):
     """Three different sequences side by side (one past length for all, as every model here batches)."""
     cfg, state, toks, _ = case(name)
     rng = np.random.default_rng(9)
-    seqs = [toks[:150], rng.integers(0, cfg["vocab"], 150).tolist(), toks[100:250]]
+    length = sum(sizes)
+    seqs = [toks[:length], rng.integers(0, cfg["vocab"], length).tolist(), toks[30:30 + length]]
     W = bm.as_numpy(state)
-    m = model_of(name, dtype, batch=3, max_prefill=64)
+    m = model_of(name, dtype, batch=3, max_prefill=max(sizes))
     got = [[] for _ in seqs]
     pos = 0
-    for n in [64, 37, 2] + [1] * 47:
+    for n in sizes:
         chunk = [s[pos:pos + n] for s in seqs]
         if n == 1:
             out = m.step([c[0] for c in chunk], pos).clone()
